@@ -6,13 +6,16 @@ from .gebadra import GebadraConfig
 from .bavetar import BavetarConfig
 from .gusorax import GusoraxConfig
 from .mobunex import MobunexConfig
+from .tuterax import TuteraxConfig
 
 register_architecture("Qwen2ForCausalLM", Qwen2Config, replace=True)
 register_architecture("Gebadra", GebadraConfig, replace=True)
 register_architecture("Bavetar", BavetarConfig, replace=True)
 register_architecture("Gusorax", GusoraxConfig, replace=True)
 register_architecture("Mobunex", MobunexConfig, replace=True)
+register_architecture("Tuterax", TuteraxConfig, replace=True)
 
 __all__ = ["BlockSpec", "ConfigError", "ModelSpec", "PartSpec", "RunStep", "Architecture",
            "architecture_name_of", "get_architecture", "known_architectures", "load_config",
-           "register_architecture", "Qwen2Config", "GebadraConfig", "BavetarConfig", "GusoraxConfig", "MobunexConfig"]
+           "register_architecture", "Qwen2Config", "GebadraConfig", "BavetarConfig", "GusoraxConfig", "MobunexConfig",
+           "TuteraxConfig"]

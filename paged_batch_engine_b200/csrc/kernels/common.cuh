@@ -51,6 +51,18 @@ __device__ __forceinline__ float block_sum(float v, float* smem /* >= 33 floats 
   return smem[32];
 }
 
+// gelu in its tanh form, 0.5 z (1 + tanh(t)) with t = sqrt(2/pi) (z + 0.044715 z^3); since
+// (1 + tanh t) / 2 = 1 / (1 + e^(-2t)) it is z times a sigmoid.  The fast form (for results that are
+// rounded to bfloat16) takes the fast exponential and division.
+__device__ __forceinline__ float gelu_tanh(float z) {
+  const float t2 = 1.5957691216057308f * fmaf(0.044715f * z * z, z, z);
+  return z / (1.0f + expf(-t2));
+}
+__device__ __forceinline__ float gelu_tanh_fast(float z) {
+  const float t2 = 1.5957691216057308f * fmaf(0.044715f * z * z, z, z);
+  return z * __fdividef(1.0f, 1.0f + __expf(-t2));
+}
+
 inline int launch_status() { return (int)cudaGetLastError(); }
 
 }  // namespace pbe

@@ -376,10 +376,11 @@ PBE_EXPORT int pbe_silu_mul(const void* in, void* out, int dtype, int rows, int 
 }
 
 // ---------------------------------------------------------------- scaled embedding + learned position row
-// out[t] = table[ids[t]] * scale + pos_table[positions[t]] (the position row unscaled), float32.
+// out[t] = table[ids[t]] * scale + pos_table[positions[t]] (the position row unscaled), float32; `lp`
+// (or null) receives a copy in bfloat16.
 template <typename TW>
-__global__ void embedding_pos_kernel(float* __restrict__ out, const TW* __restrict__ table,
-                                     const int32_t* __restrict__ ids, float scale, const TW* __restrict__ pos_table,
+__global__ void embedding_pos_kernel(float* __restrict__ out, __nv_bfloat16* __restrict__ lp,
+                                     const TW* __restrict__ table, const int32_t* __restrict__ ids, float scale, const TW* __restrict__ pos_table,
                                      const int32_t* __restrict__ positions, int max_pos, int d, int vocab) {
   pdl_launch_dependents();
   pdl_wait();
@@ -394,19 +395,20 @@ __global__ void embedding_pos_kernel(float* __restrict__ out, const TW* __restri
     float v = ok ? to_float(row[i]) * scale : 0.f;
     if (prow) v += to_float(prow[i]);
     o[i] = v;
+    if (lp) lp[(size_t)t * d + i] = __float2bfloat16_rn(v);
   }
 }
 
-PBE_EXPORT int pbe_embedding_pos(float* out, const void* table, int table_dtype, const int32_t* ids, float scale,
+PBE_EXPORT int pbe_embedding_pos(float* out, void* lp, const void* table, int table_dtype, const int32_t* ids, float scale,
                                  const void* pos_table, const int32_t* positions, int max_pos, int num_tokens,
                                  int d, int vocab, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
   const int threads = d >= 1024 ? 256 : 128;
   if (table_dtype == PBE_F32)
-    launch_k(embedding_pos_kernel<float>, num_tokens, threads, 0, stream, out, (const float*)table, ids, scale,
+    launch_k(embedding_pos_kernel<float>, num_tokens, threads, 0, stream, out, (__nv_bfloat16*)lp, (const float*)table, ids, scale,
              (const float*)pos_table, positions, max_pos, d, vocab);
   else
-    launch_k(embedding_pos_kernel<__nv_bfloat16>, num_tokens, threads, 0, stream, out, (const __nv_bfloat16*)table,
+    launch_k(embedding_pos_kernel<__nv_bfloat16>, num_tokens, threads, 0, stream, out, (__nv_bfloat16*)lp, (const __nv_bfloat16*)table,
              ids, scale, (const __nv_bfloat16*)pos_table, positions, max_pos, d, vocab);
   return launch_status();
 }
@@ -448,6 +450,7 @@ PBE_EXPORT int pbe_fold_pair(const float* residual, const void* delta_a, const v
 // ---------------------------------------------------------------- gated activations other than silu(g) * u
 // in: [rows, 2*inter], gate in columns [0, inter), linear part in [inter, 2*inter); out [rows, inter].
 // kind 1 (capped swish): g <- min(g, limit), u <- clamp(u, -limit, limit), y = g * sigmoid(alpha * g) * (u + 1).
+// kind 2 (gelu, tanh form): y = gelu_tanh(g) * u.
 template <typename T>
 __global__ void glu_act_kernel(const T* __restrict__ in, T* __restrict__ out, int inter, size_t total, int kind,
                                float limit, float alpha) {
@@ -464,6 +467,8 @@ __global__ void glu_act_kernel(const T* __restrict__ in, T* __restrict__ out, in
       g = fminf(g, limit);
       u = fminf(fmaxf(u, -limit), limit);
       y = (g / (1.0f + expf(-alpha * g))) * (u + 1.0f);
+    } else if (kind == 2) {
+      y = gelu_tanh(g) * u;
     } else {
       y = (g / (1.0f + expf(-g))) * u;
     }
@@ -503,13 +508,42 @@ __global__ void capped_swish_bf16x8_kernel(const __nv_bfloat16* __restrict__ in,
   }
 }
 
+// gelu_tanh(g) * u on bfloat16 rows, eight values a thread
+__global__ void gelu_mul_bf16x8_kernel(const __nv_bfloat16* __restrict__ in, __nv_bfloat16* __restrict__ out, int inter,
+                                       int rows) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int chunk = blockIdx.x * blockDim.x + threadIdx.x;
+  if (chunk * 8 >= inter) return;
+  for (int r = blockIdx.y; r < rows; r += gridDim.y) {
+    const __nv_bfloat16* row = in + (size_t)r * 2 * inter;
+    const uint4 gq = *reinterpret_cast<const uint4*>(row + chunk * 8);
+    const uint4 uq = *reinterpret_cast<const uint4*>(row + inter + chunk * 8);
+    const unsigned gw[4] = {gq.x, gq.y, gq.z, gq.w}, uw[4] = {uq.x, uq.y, uq.z, uq.w};
+    unsigned yw[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float2 g = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gw[i]));
+      const float2 u = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&uw[i]));
+      const __nv_bfloat162 y = __floats2bfloat162_rn(gelu_tanh_fast(g.x) * u.x, gelu_tanh_fast(g.y) * u.y);
+      yw[i] = *reinterpret_cast<const unsigned*>(&y);
+    }
+    *reinterpret_cast<uint4*>(out + (size_t)r * inter + chunk * 8) = make_uint4(yw[0], yw[1], yw[2], yw[3]);
+  }
+}
+
 PBE_EXPORT int pbe_glu_act(const void* in, void* out, int dtype, int rows, int inter, int kind, float limit,
                            float alpha, cudaStream_t stream) {
   const size_t total = (size_t)rows * inter;
   if (total == 0) return 0;
-  if (kind == 1 && dtype == PBE_BF16 && (inter & 7) == 0 && (((uintptr_t)in | (uintptr_t)out) & 15) == 0) {
+  if (kind != 0 && dtype == PBE_BF16 && (inter & 7) == 0 && (((uintptr_t)in | (uintptr_t)out) & 15) == 0) {
     const int threads = 256, chunks = inter / 8;
     dim3 grid((chunks + threads - 1) / threads, rows < 65535 ? rows : 65535);
+    if (kind == 2) {
+      launch_k(gelu_mul_bf16x8_kernel, grid, threads, 0, stream, (const __nv_bfloat16*)in, (__nv_bfloat16*)out, inter,
+               rows);
+      return launch_status();
+    }
     launch_k(capped_swish_bf16x8_kernel, grid, threads, 0, stream, (const __nv_bfloat16*)in, (__nv_bfloat16*)out,
              inter, rows, limit, alpha);
     return launch_status();

@@ -57,6 +57,7 @@ struct StreamParams {
   int ld_y;
   int up_offset;       // row of W where the up rows start (SwiGLU)
   int y_float;         // 1: float32 output
+  int glu;             // the gated epilogue's activation: 0 silu, 1 gelu (tanh form)
   int mb;              // batch rows of the MMA: M rounded up to 16
   int tiles_n;         // tiles of 128 output columns
   int splits;          // K splits a tile
@@ -255,7 +256,8 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_const
           else ((bf16*)p.Y)[(size_t)m * p.ld_y + n] = __float2bfloat16_rn(val);
         }
       };
-      auto silu_mul = [](float g, float u) {     // as the bfloat16 silu_mul kernel does
+      auto act_mul = [&](float g, float u) {     // as the bfloat16 activation kernels do
+        if (p.glu) return gelu_tanh_fast(g) * u;
         return (g * __fdividef(1.0f, 1.0f + __expf(-g))) * u;
       };
       for (int c = 0; c < chunks; ++c) {
@@ -265,7 +267,7 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_const
         if (direct) {
           if (n < p.N_out) {
 #pragma unroll
-            for (int i = 0; i < 16; ++i) put(c * 16 + i, SWIGLU ? silu_mul(v[i], u[i]) : v[i]);
+            for (int i = 0; i < 16; ++i) put(c * 16 + i, SWIGLU ? act_mul(v[i], u[i]) : v[i]);
           }
         } else {
 #pragma unroll
@@ -309,7 +311,7 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_const
             }
           }
 #pragma unroll
-          for (int i = 0; i < 16; ++i) put(c * 16 + i, SWIGLU ? silu_mul(a[i], b[i]) : a[i]);
+          for (int i = 0; i < 16; ++i) put(c * 16 + i, SWIGLU ? act_mul(a[i], b[i]) : a[i]);
         }
       }
       if (threadIdx.x == 64) p.tickets[tile] = 0;      // ready for the next launch
@@ -377,15 +379,19 @@ PBE_EXPORT long long pbe_gemm_stream_scratch_floats(int M, int N, int K, int mod
   return (long long)splits * tiles_n * W_ROWS * mb * (mode == 1 ? 2 : 1);
 }
 
-// mode 0: Y[M, N] = X W^T; mode 1: W is [gate; up] with N rows in total, Y[M, N/2] = silu(X gate^T) * (X up^T).
+// mode 0: Y[M, N] = X W^T; mode 1: W is [gate; up] with N rows in total, Y[M, N/2] = silu(X gate^T) * (X up^T);
+// mode 3: the same with gelu (tanh form) for silu.
 // err: device int, set to 1 if a bounded wait ran out (the result is then invalid).
 PBE_EXPORT int pbe_gemm_stream(const void* X, const void* W, void* Y, int y_dtype, int M, int N, int K, int mode,
                                float* scratch, int* tickets, int* err, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (M > MAX_ROWS || K <= 0 || (K & 7) != 0) return (int)cudaErrorInvalidValue;      // TMA: row stride a multiple of 16 bytes
   if (((uintptr_t)X & 15) || ((uintptr_t)W & 15)) return (int)cudaErrorInvalidValue;
+  const int glu = mode == 3 ? 1 : 0;
+  if (mode == 3) mode = 1;
   if (mode == 1 && ((N & 1) || y_dtype != PBE_BF16)) return (int)cudaErrorInvalidValue;
   StreamParams p;
+  p.glu = glu;
   p.Y = Y;
   p.M = M;
   p.K = K;

@@ -5,12 +5,20 @@
 //     row's own chunk of C positions (chunks counted from position 0 of the sequence);
 //   * a bias per (head, distance) added to the scaled score: bias[h][min(i - j, rows - 1)], a table
 //     the host expands from whatever rule the model has (buckets, slopes ...);
-//   * a unit sink: one more term e^0 in the softmax's denominator that carries no value;
+//   * a cap on the scaled score, c tanh(s / c);
+//   * a sink: one more term in the softmax's denominator that carries no value, e^0 or e^(a learned
+//     number of the head);
+//   * values that were rotated by their position when they were cached: each head's output is turned
+//     back by the row's position, pair by pair (e with e + E / 2), before the gate;
 //   * a gate: the output of head h, element e, times sigmoid(gate[t][h * E + e]).
 //
 // head_norm_write: per token, the projection's bias, an RMS norm over each head's D query or key
 //   elements with one gain vector shared by the heads (float32 throughout), optionally a factor per
-//   query head (a learned temperature), queries out in float32, keys and values into the pages.
+//   query head (a learned temperature), a rotation of the first rot_dims dimensions of queries and
+//   keys and one of whole values (halves paired: i with i + half), queries out in float32, keys and
+//   values into the pages.  The angle's fraction of a turn is formed from the frequency as two
+//   float32 numbers and the exact remainder of the product, so it is good to a few 1e-8 of a turn at
+//   any position.  cos and sin of the values' angles are left in a table for the attention's epilogue.
 // masked_attention: the float32-arithmetic kernel.  It reads the engine's attention work list
 //   (request, row tile, key split, splits): the rows of a request are packed with the query heads
 //   that share a key/value head, 16 packed rows a block, 32 keys a tile (a key a lane), online
@@ -40,15 +48,46 @@ struct HeadNormParams {
   void* v_pages;             // [page][G][page_tokens][E]
   int H, G, D, E, page_tokens;
   float eps;
+  const int32_t* positions;  // [T], read when something turns
+  const float2* rot_freq;    // [rot_dims / 2] turns a position as (rounded, rest), or null: no rotation of q and k
+  int rot_dims;
+  const float2* v_freq;      // [E / 2] the same for values, or null
+  float2* v_turn;            // [T, E / 2] (cos, sin) of the values' angles, written when v_freq is given
 };
+
+// (cos, sin) of 2 pi * position * freq
+__device__ __forceinline__ float2 turn_of(int position, float2 freq) {
+  const float p = (float)position;               // exact up to 2^24
+  const float whole = rintf(p * freq.x);
+  const float rest = fmaf(p, freq.x, -whole) + p * freq.y;
+  float2 cs;
+  sincospif(2.0f * rest, &cs.y, &cs.x);
+  return cs;
+}
 
 constexpr int HN_MAX = 8;    // elements of a head a lane holds at most (D <= 256)
 
-template <typename T>
+template <typename T, bool TURN>
 __global__ void __launch_bounds__(128) head_norm_write_kernel(HeadNormParams p) {
+  __shared__ float2 rot_cs[TURN ? 16 * HN_MAX : 1], v_cs[TURN ? 16 * HN_MAX : 1];   // heads are at most 256 wide
+  __shared__ float held[TURN ? 4 : 1][TURN ? 32 * HN_MAX : 1];     // a warp's head between the norm and the turn
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
+  if (TURN) {
+    const int half = p.rot_freq ? p.rot_dims / 2 : 0, vhalf = p.v_freq ? p.E / 2 : 0;
+    const int pos = p.positions[t];
+    for (int i = threadIdx.x; i < half + vhalf; i += blockDim.x) {
+      if (i < half) {
+        rot_cs[i] = turn_of(pos, p.rot_freq[i]);
+      } else {
+        const float2 cs = turn_of(pos, p.v_freq[i - half]);
+        v_cs[i - half] = cs;
+        p.v_turn[(size_t)t * vhalf + i - half] = cs;
+      }
+    }
+    __syncthreads();
+  }
   const int H = p.H, G = p.G, D = p.D, E = p.E, PT = p.page_tokens;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const T* row = (const T*)p.proj + (size_t)t * p.ld;
@@ -74,18 +113,51 @@ __global__ void __launch_bounds__(128) head_norm_write_kernel(HeadNormParams p) 
     }
     float sc = 1.f;
     if (gain) sc = 1.0f / sqrtf(warp_sum(ss) / (float)D + p.eps);
+    const int half = (TURN && p.rot_freq) ? p.rot_dims / 2 : 0;
+    if (half) {
+      __syncwarp();                            // the warp's head before is read
+#pragma unroll
+      for (int i = 0; i < HN_MAX; ++i) {
+        const int d = lane + i * 32;
+        if (d < D) {
+          x[i] = gain ? (x[i] * sc) * gain[d] : x[i];
+          if (d < 2 * half) held[TURN ? warp : 0][TURN ? d : 0] = x[i];
+        }
+      }
+      __syncwarp();
+    }
 #pragma unroll
     for (int i = 0; i < HN_MAX; ++i) {
       const int d = lane + i * 32;
       if (d < D) {
-        float y = gain ? (x[i] * sc) * gain[d] : x[i];
+        float y = (gain && !half) ? (x[i] * sc) * gain[d] : x[i];
+        if (d < 2 * half) {
+          const bool first = d < half;
+          const float other = held[TURN ? warp : 0][TURN ? (first ? d + half : d - half) : 0];
+          const float2 cs = rot_cs[TURN ? (first ? d : d - half) : 0];
+          y = first ? y * cs.x - other * cs.y : y * cs.x + other * cs.y;
+        }
         if (is_q && p.q_head_scale) y *= p.q_head_scale[head];
         if (is_q) p.q_out[((size_t)t * H + head) * D + d] = y;
         else ((T*)p.k_pages)[(((size_t)page * G + head) * PT + off) * D + d] = from_float<T>(y);
       }
     }
   }
-  if (store && p.v_pages) {
+  if (TURN && store && p.v_pages && p.v_freq) {
+    const int vhalf = E / 2;
+    for (int i = threadIdx.x; i < G * vhalf; i += blockDim.x) {
+      const int head = i / vhalf, m = i - head * vhalf, c = p.v_off + head * E + m;
+      float u = to_float(row[c]), v = to_float(row[c + vhalf]);
+      if (p.bias) {
+        u += p.bias[c];
+        v += p.bias[c + vhalf];
+      }
+      const float2 cs = v_cs[m];
+      T* dst = (T*)p.v_pages + (((size_t)page * G + head) * PT + off) * E + m;
+      dst[0] = from_float<T>(u * cs.x - v * cs.y);
+      dst[vhalf] = from_float<T>(v * cs.x + u * cs.y);
+    }
+  } else if (store && p.v_pages) {
     for (int i = threadIdx.x; i < G * E; i += blockDim.x) {
       const int head = i / E, e = i - head * E;
       const float y = to_float(row[p.v_off + i]) + (p.bias ? p.bias[p.v_off + i] : 0.f);
@@ -248,6 +320,7 @@ __global__ void __launch_bounds__(NWARPS * 32) masked_attention_kernel(AttnParam
       float sc = -INFINITY;
       if (visible) {
         sc = s[j] * p.scale;
+        if (x.softcap > 0.f) sc = x.softcap * tanhf(sc / x.softcap);
         if (x.bias) sc += __ldg(x.bias + (size_t)row_head[j] * x.bias_rows + min(pos - key, x.bias_rows - 1));
       }
       const float m_new = fmaxf(m_run[j], warp_max(sc));
@@ -275,6 +348,7 @@ __global__ void __launch_bounds__(NWARPS * 32) masked_attention_kernel(AttnParam
     }
   }
 
+  if (x.turn) __syncthreads();     // the values are read: their place holds a row of outputs a warp while it turns
 #pragma unroll
   for (int j = 0; j < ROWS_PER_WARP; ++j) {
     const int pr = pr0 + warp + j * NWARPS;
@@ -284,15 +358,32 @@ __global__ void __launch_bounds__(NWARPS * 32) masked_attention_kernel(AttnParam
     const int t = qs + row;
     if (nsplit <= 1) {
       float m = m_run[j], l = l_run[j], rescale = 1.f;
-      if (x.unit_sink) add_unit_sink(m, l, rescale);
+      if (x.has_sink) add_sink(m, l, rescale, x.sink ? x.sink[head] : 0.f);
       const float inv = l > 0.f ? rescale / l : 0.f;
       T* o = (T*)p.out + ((size_t)t * H + head) * E;
       const T* g = x.gate ? (const T*)x.gate + (size_t)t * x.ldg + head * E : nullptr;
+      float* held = Vs + warp * E;
+      const int half = E / 2;
+      if (x.turn) {
+        __syncwarp();
+#pragma unroll
+        for (int ii = 0; ii < EPL; ++ii) {
+          const int e = lane + ii * 32;
+          if (e < E) held[e] = acc[j][ii] * inv;
+        }
+        __syncwarp();
+      }
 #pragma unroll
       for (int ii = 0; ii < EPL; ++ii) {
         const int e = lane + ii * 32;
         if (e < E) {
           float y = acc[j][ii] * inv;
+          if (x.turn) {
+            const bool first = e < half;
+            const float2 cs = x.turn[(size_t)t * half + (first ? e : e - half)];
+            const float other = held[first ? e + half : e - half];
+            y = first ? y * cs.x + other * cs.y : y * cs.x - other * cs.y;
+          }
           if (g) y *= sigmoidf_(to_float(g[e]));
           o[e] = from_float<T>(y);
         }
@@ -315,7 +406,9 @@ __global__ void __launch_bounds__(NWARPS * 32) masked_attention_kernel(AttnParam
 }
 
 struct MaskedMergeExtra {
-  int unit_sink;
+  int has_sink;
+  const float* sink;
+  const float2* turn;
   const void* gate;
   int ldg;
 };
@@ -332,8 +425,9 @@ __global__ void masked_merge_kernel(AttnMergeParams p, MaskedMergeExtra x) {
   const size_t base = ((size_t)srow * p.num_heads + head) * p.max_splits;
   float m = -INFINITY;
   for (int s = 0; s < n; ++s) m = fmaxf(m, p.part_ml[(base + s) * 2]);
-  if (x.unit_sink) m = fmaxf(m, 0.f);
-  float l = x.unit_sink ? expf(-m) : 0.f;
+  const float s_sink = (x.has_sink && x.sink) ? x.sink[head] : 0.f;
+  if (x.has_sink) m = fmaxf(m, s_sink);
+  float l = x.has_sink ? expf(s_sink - m) : 0.f;
   for (int s = 0; s < n; ++s) {
     const float ms = p.part_ml[(base + s) * 2];
     if (ms != -INFINITY) l += p.part_ml[(base + s) * 2 + 1] * expf(ms - m);
@@ -341,13 +435,30 @@ __global__ void masked_merge_kernel(AttnMergeParams p, MaskedMergeExtra x) {
   const float inv = l > 0.f ? 1.0f / l : 0.f;
   T* o = (T*)p.out + ((size_t)t * p.num_heads + head) * E;
   const T* g = x.gate ? (const T*)x.gate + (size_t)t * x.ldg + head * E : nullptr;
-  for (int e = threadIdx.x; e < E; e += blockDim.x) {
+  auto sum_at = [&](int e) {
     float a = 0.f;
     for (int s = 0; s < n; ++s) {
       const float ms = p.part_ml[(base + s) * 2];
       if (ms != -INFINITY) a += p.part_o[(base + s) * E + e] * expf(ms - m);
     }
-    float y = a * inv;
+    return a * inv;
+  };
+  if (x.turn) {
+    const int half = E / 2;
+    for (int e = threadIdx.x; e < half; e += blockDim.x) {
+      float u = sum_at(e), v = sum_at(e + half);
+      turn_back(u, v, x.turn[(size_t)t * half + e]);
+      if (g) {
+        u *= sigmoidf_(to_float(g[e]));
+        v *= sigmoidf_(to_float(g[e + half]));
+      }
+      o[e] = from_float<T>(u);
+      o[e + half] = from_float<T>(v);
+    }
+    return;
+  }
+  for (int e = threadIdx.x; e < E; e += blockDim.x) {
+    float y = sum_at(e);
     if (g) y *= sigmoidf_(to_float(g[e]));
     o[e] = from_float<T>(y);
   }
@@ -386,35 +497,46 @@ PBE_EXPORT int pbe_head_norm_write(const void* proj, int ld, int q_off, int k_of
                                    const float* q_gain, const float* k_gain, const float* q_head_scale,
                                    const int32_t* slots, float* q_out,
                                    void* k_pages, void* v_pages, int T, int H, int G, int D, int E, int page_tokens,
-                                   float eps, int dtype, cudaStream_t stream) {
+                                   float eps, const int32_t* positions, const float2* rot_freq, int rot_dims,
+                                   const float2* v_freq, float2* v_turn, int dtype, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (D > 32 * HN_MAX || D < 1 || E < 1) return (int)cudaErrorInvalidValue;
+  const bool turns = rot_freq != nullptr || v_freq != nullptr;
+  if (turns && positions == nullptr) return (int)cudaErrorInvalidValue;
+  if (rot_freq && (rot_dims < 2 || (rot_dims & 1) || rot_dims > D)) return (int)cudaErrorInvalidValue;
+  if (v_freq && (v_turn == nullptr || (E & 1) || E > 32 * HN_MAX)) return (int)cudaErrorInvalidValue;
   HeadNormParams p{proj, ld, q_off, k_off, v_off, bias, q_gain, k_gain, q_head_scale, slots, q_out, k_pages, v_pages,
-                   H, G, D, E, page_tokens, eps};
-  if (dtype == PBE_F32) launch_k(head_norm_write_kernel<float>, T, 128, 0, stream, p);
-  else launch_k(head_norm_write_kernel<__nv_bfloat16>, T, 128, 0, stream, p);
+                   H, G, D, E, page_tokens, eps, positions, rot_freq, rot_dims, v_freq, v_turn};
+  if (dtype == PBE_F32) {
+    if (turns) launch_k(head_norm_write_kernel<float, true>, T, 128, 0, stream, p);
+    else launch_k(head_norm_write_kernel<float, false>, T, 128, 0, stream, p);
+  } else {
+    if (turns) launch_k(head_norm_write_kernel<__nv_bfloat16, true>, T, 128, 0, stream, p);
+    else launch_k(head_norm_write_kernel<__nv_bfloat16, false>, T, 128, 0, stream, p);
+  }
   return launch_status();
 }
 
 PBE_EXPORT int pbe_masked_attention(const AttnParams* params, int D, int E, const float* bias, int bias_rows,
-                                    int mask_kind, int unit_sink, const void* gate, int ldg, int num_work,
-                                    int dtype, cudaStream_t stream) {
+                                    int mask_kind, int has_sink, const float* sink, float softcap,
+                                    const float2* turn, const void* gate, int ldg, int num_work, int dtype,
+                                    cudaStream_t stream) {
   if (num_work <= 0) return 0;
   AttnParams p = *params;
   if (p.num_heads % p.num_kv_heads != 0 || p.tile_rows != BM || p.split_keys % BN != 0 || D < 1 || E < 1 ||
-      E > 256 || mask_kind < 0 || mask_kind > 2 || (mask_kind != 0 && p.window < 1) || (bias && bias_rows < 1))
+      E > 256 || (turn && (E & 1)) || mask_kind < 0 || mask_kind > 2 || (mask_kind != 0 && p.window < 1) || (bias && bias_rows < 1))
     return (int)cudaErrorInvalidValue;
   if (ma_smem(D, E) > 200 * 1024) return (int)cudaErrorInvalidValue;
-  MaskedExtra x{bias, bias_rows, mask_kind, unit_sink, gate, ldg, D, E};
+  MaskedExtra x{bias, bias_rows, mask_kind, has_sink, sink, softcap, turn, gate, ldg, D, E};
   return dtype == PBE_F32 ? dispatch_ma<float>(p, x, num_work, stream)
                           : dispatch_ma<__nv_bfloat16>(p, x, num_work, stream);
 }
 
-PBE_EXPORT int pbe_masked_merge(const AttnMergeParams* params, int unit_sink, const void* gate, int ldg,
-                                int split_rows, int dtype, cudaStream_t stream) {
+PBE_EXPORT int pbe_masked_merge(const AttnMergeParams* params, int has_sink, const float* sink, const float2* turn,
+                                const void* gate, int ldg, int split_rows, int dtype, cudaStream_t stream) {
   if (split_rows <= 0) return 0;
   AttnMergeParams p = *params;
-  MaskedMergeExtra x{unit_sink, gate, ldg};
+  MaskedMergeExtra x{has_sink, sink, turn, gate, ldg};
   dim3 grid(split_rows, p.num_heads);
   const int threads = p.head_dim > 64 ? 128 : 64;
   if (dtype == PBE_F32) launch_k(masked_merge_kernel<float>, grid, threads, 0, stream, p, x);

@@ -1,8 +1,8 @@
 // The masked attention of masked_attention.cu for bfloat16 pages on the tensor cores (mma.sync
 // m16n8k16, float32 accumulation), flash style: scores, softmax statistics and the output
 // accumulator stay in registers; keys and values stream from the pages through shared memory,
-// double buffered with cp.async.  Same options (mask, bias by head and distance, unit sink, gate),
-// same work list (request, row tile, key split) and the same partial buffers as the float32 kernel,
+// double buffered with cp.async.  Same options (mask, score cap, bias by head and distance, sink,
+// turned-back outputs, gate), same work list (request, row tile, key split) and the same partial buffers as the float32 kernel,
 // whose merge kernel puts the key splits together.
 //
 // Scores and softmax weights are float32 quantities and stay so through the tensor cores: the
@@ -97,6 +97,15 @@ __device__ __forceinline__ void split_pair(float x, float y, unsigned& hi, unsig
   const float xh = __uint_as_float(hi << 16), yh = __uint_as_float(hi & 0xffff0000u);
   const __nv_bfloat162 l = __floats2bfloat162_rn(x - xh, y - yh);
   lo = *reinterpret_cast<const unsigned*>(&l);
+}
+
+// c * tanh(s) with the argument given as e^(2 s) = 2^z: c - 2 c / (1 + 2^z).  The hardware's exponential
+// and reciprocal are good to two units in the last place, so the result is to about 1e-7 of c.
+__device__ __forceinline__ float capped(float z, float c) {
+  float e, r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(z));
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
+  return fmaf(-2.0f * c, r, c);
 }
 
 __global__ void __launch_bounds__(NT, PBE_MA_BLOCKS) masked_attention_mma_kernel(AttnParams p, MaskedExtra x) {
@@ -276,13 +285,23 @@ __global__ void __launch_bounds__(NT, PBE_MA_BLOCKS) masked_attention_mma_kernel
       }
       // scale, bias, mask; the tile's row maxima
       float mx[2] = {-INFINITY, -INFINITY};
+      float scale = p.scale;
+      if (x.softcap > 0.f) {
+        // capped scores first; what follows then has nothing to scale
+        const float z = p.scale * (2.885390081777927f / x.softcap);       // 2 log2(e) / c
+#pragma unroll
+        for (int nt = 0; nt < SNT; ++nt)
+#pragma unroll
+          for (int c = 0; c < 4; ++c) S[nt][c] = capped(S[nt][c] * z, x.softcap);
+        scale = 1.0f;
+      }
       if (!keys_mode && tk >= all_lo && tk + kwidth - 1 <= all_hi) {
         // every row of the warp sees every key of its part of the tile
 #pragma unroll
         for (int nt = 0; nt < SNT; ++nt) {
 #pragma unroll
           for (int c = 0; c < 4; ++c) {
-            const float sc = x.bias ? fmaf(S[nt][c], p.scale, B[nt][c]) : S[nt][c] * p.scale;
+            const float sc = x.bias ? fmaf(S[nt][c], scale, B[nt][c]) : S[nt][c] * scale;
             S[nt][c] = sc;
             mx[c >> 1] = fmaxf(mx[c >> 1], sc);
           }
@@ -297,7 +316,7 @@ __global__ void __launch_bounds__(NT, PBE_MA_BLOCKS) masked_attention_mma_kernel
             const int key = tk + nt * 8 + 2 * t + (c & 1);
             float sc = -INFINITY;
             if (!skip && key >= lo[i] && key <= hi[i])
-              sc = x.bias ? fmaf(S[nt][c], p.scale, B[nt][c]) : S[nt][c] * p.scale;
+              sc = x.bias ? fmaf(S[nt][c], scale, B[nt][c]) : S[nt][c] * scale;
             S[nt][c] = sc;
             mx[i] = fmaxf(mx[i], sc);
           }
@@ -413,8 +432,18 @@ __global__ void __launch_bounds__(NT, PBE_MA_BLOCKS) masked_attention_mma_kernel
     const int tok = qs + (pos[i] - pos0);
     if (nsplit <= 1) {
       float m = m_run[i], l = l_run[i], rescale = 1.f;
-      if (x.unit_sink) add_unit_sink(m, l, rescale);
+      if (x.has_sink) add_sink(m, l, rescale, x.sink ? x.sink[head[i]] : 0.f);
       const float inv = l > 0.f ? rescale / l : 0.f;
+      if (x.turn) {
+        // the values' pairs (e, e + E / 2) lie in one thread's registers
+        const float2* cs = x.turn + (size_t)tok * (E / 2);
+#pragma unroll
+        for (int on = 0; on < ONT / 2; ++on) {
+          const float4 c2 = *reinterpret_cast<const float4*>(cs + on * 8 + 2 * t);
+          turn_back(O[on][2 * i], O[on + ONT / 2][2 * i], make_float2(c2.x, c2.y));
+          turn_back(O[on][2 * i + 1], O[on + ONT / 2][2 * i + 1], make_float2(c2.z, c2.w));
+        }
+      }
       bf16* o = (bf16*)p.out + ((size_t)tok * H + head[i]) * E;
       const bf16* gt = x.gate ? (const bf16*)x.gate + (size_t)tok * x.ldg + head[i] * E : nullptr;
       // the row's gate values are all requested before the first store (a store could alias them
@@ -462,15 +491,15 @@ PBE_EXPORT int pbe_masked_attention_mma_tile_rows() { return BM; }
 PBE_EXPORT int pbe_masked_attention_mma_key_tile() { return BN; }
 
 PBE_EXPORT int pbe_masked_attention_mma(const AttnParams* params, const float* bias, int bias_rows, int mask_kind,
-                                        int unit_sink, const void* gate, int ldg, int num_work,
-                                        cudaStream_t stream) {
+                                        int has_sink, const float* sink, float softcap, const float2* turn,
+                                        const void* gate, int ldg, int num_work, cudaStream_t stream) {
   if (num_work <= 0) return 0;
   AttnParams p = *params;
   if (p.num_heads % p.num_kv_heads != 0 || p.tile_rows != BM || p.split_keys % BN != 0 || mask_kind < 0 ||
       mask_kind > 2 || (mask_kind != 0 && p.window < 1) || (bias && bias_rows < 1))
     return (int)cudaErrorInvalidValue;
   // rows are fetched in 16-byte pieces
-  if ((((uintptr_t)p.q | (uintptr_t)p.k_cache | (uintptr_t)p.v_cache | (uintptr_t)p.part_o) & 15) != 0 ||
+  if ((((uintptr_t)p.q | (uintptr_t)turn | (uintptr_t)p.k_cache | (uintptr_t)p.v_cache | (uintptr_t)p.part_o) & 15) != 0 ||
       ((uintptr_t)p.out & 3) != 0)
     return (int)cudaErrorMisalignedAddress;
   static bool opted = false;
@@ -480,7 +509,7 @@ PBE_EXPORT int pbe_masked_attention_mma(const AttnParams* params, const float* b
     if (e != cudaSuccess) return (int)e;
     opted = true;
   }
-  MaskedExtra x{bias, bias_rows, mask_kind, unit_sink, gate, ldg, D, E};
+  MaskedExtra x{bias, bias_rows, mask_kind, has_sink, sink, softcap, turn, gate, ldg, D, E};
   x.gate_pairs = gate != nullptr && ((uintptr_t)gate & 3) == 0 && (ldg & 1) == 0;
   launch_k(masked_attention_mma_kernel, dim3(num_work, p.num_kv_heads), NT, SMEM_BYTES, stream, p, x);
   return launch_status();

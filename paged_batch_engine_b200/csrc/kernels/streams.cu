@@ -153,6 +153,7 @@ struct GatedRmsParams {
   float eps;
   int per_head;            // 1: each head's E values have a root mean square of their own
   int gate_act;            // 0: sigmoid, 1: silu
+  int gate_f32;            // 1: the gate is float32 whatever the output is
   int gate_first;          // 1: the gate multiplies o before the root mean square is taken (of the gated values)
 };
 
@@ -164,9 +165,10 @@ __global__ void gated_rms_kernel(GatedRmsParams p) {
   const int t = blockIdx.x, H = p.H, E = p.E, N = H * E;
   const float* o = p.o + (size_t)t * N;
   const T* g = (const T*)p.gate + (size_t)t * p.ld_gate;
+  const float* gf = (const float*)p.gate + (size_t)t * p.ld_gate;
   T* out = (T*)p.out + (size_t)t * N;
   auto gate_of = [&](int c) {
-    const float gv = to_float(g[c]);
+    const float gv = p.gate_f32 ? gf[c] : to_float(g[c]);
     const float sg = 1.0f / (1.0f + expf(-gv));
     return p.gate_act ? gv * sg : sg;
   };
@@ -245,11 +247,11 @@ PBE_EXPORT int pbe_branch_rms_mean(const void* const* x, const float* const* gai
   return launch_status();
 }
 
-PBE_EXPORT int pbe_gated_rms(const float* o, const void* gate, int ld_gate, const float* gain, void* out, int dtype,
+PBE_EXPORT int pbe_gated_rms(const float* o, const void* gate, int gate_dtype, int ld_gate, const float* gain, void* out, int dtype,
                              int T, int H, int E, float eps, int per_head, int gate_act, int gate_first,
                              cudaStream_t stream) {
   if (T <= 0) return 0;
-  GatedRmsParams p{o, gate, gain, out, ld_gate, H, E, eps, per_head, gate_act, gate_first};
+  GatedRmsParams p{o, gate, gain, out, ld_gate, H, E, eps, per_head, gate_act, gate_dtype == PBE_F32 ? 1 : 0, gate_first};
   const int threads = H * E >= 512 ? 256 : 128;
   if (dtype == PBE_F32) launch_k(gated_rms_kernel<float>, T, threads, 0, stream, p);
   else launch_k(gated_rms_kernel<__nv_bfloat16>, T, threads, 0, stream, p);

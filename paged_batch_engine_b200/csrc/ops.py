@@ -7,6 +7,7 @@ a CUDA device is an error, and so is a failed build of the kernel library.
 from __future__ import annotations
 
 import ctypes
+import math
 import os
 from typing import Optional
 
@@ -109,9 +110,11 @@ def embedding(out: torch.Tensor, table: torch.Tensor, ids: torch.Tensor) -> torc
 
 
 def embedding_positions(out: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, scale: float,
-                        pos_table: Optional[torch.Tensor], positions: Optional[torch.Tensor]) -> torch.Tensor:
+                        pos_table: Optional[torch.Tensor], positions: Optional[torch.Tensor],
+                        lp_dtype: Optional[torch.dtype] = None) -> Optional[torch.Tensor]:
     """out[t, :] = table[ids[t], :] * scale + pos_table[positions[t], :] as float32 (the position row is
-    not scaled; ``pos_table`` None: no position row)."""
+    not scaled; ``pos_table`` None: no position row).  Returns a copy of the rows in ``lp_dtype``
+    (bfloat16), or None when that is None."""
     _need_cuda(out, table, ids, pos_table, positions)
     _need_contiguous(out, table, ids, pos_table, positions)
     if out.dtype != torch.float32 or ids.dtype != torch.int32:
@@ -122,11 +125,15 @@ def embedding_positions(out: torch.Tensor, table: torch.Tensor, ids: torch.Tenso
     if pos_table is not None and (pos_table.dtype != table.dtype or pos_table.shape[1] != d or positions is None
                                   or positions.dtype != torch.int32 or positions.numel() != T):
         raise KernelError("embedding: the position table has the embedding's dtype and width, positions are int32 [T]")
+    if lp_dtype not in (None, torch.bfloat16):
+        raise KernelError("embedding: the copy is bfloat16")
+    lp = torch.empty((T, d), dtype=lp_dtype, device=out.device) if lp_dtype is not None else None
     fn = _fn("elementwise", "pbe_embedding_pos",
-             [c_void_p, c_void_p, c_int, c_void_p, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
-    _check(fn(_ptr(out), _ptr(table), _dtype_code(table), _ptr(ids), float(scale), _ptr(pos_table), _ptr(positions),
+             [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+              c_void_p])
+    _check(fn(_ptr(out), _ptr(lp), _ptr(table), _dtype_code(table), _ptr(ids), float(scale), _ptr(pos_table), _ptr(positions),
               pos_table.shape[0] if pos_table is not None else 0, T, d, table.shape[0], _stream()), "embedding_pos")
-    return out
+    return lp
 
 
 def fold_pair(residual: torch.Tensor, delta_a: Optional[torch.Tensor], delta_b: Optional[torch.Tensor],
@@ -151,13 +158,15 @@ def fold_pair(residual: torch.Tensor, delta_a: Optional[torch.Tensor], delta_b: 
     return out
 
 
-GLU_ACTIVATIONS = {"silu": 0, "capped_swish": 1}
+GLU_ACTIVATIONS = {"silu": 0, "capped_swish": 1, "gelu_tanh": 2}
+GLU_EPILOGUES = {"silu": 1, "gelu_tanh": 3}      # those the few-row products have as an epilogue, and their mode
 
 
 def gated_activation(gate_up: torch.Tensor, out: torch.Tensor, activation: str = "silu", limit: float = 0.0,
                      alpha: float = 1.0) -> torch.Tensor:
     """out[r, c] = act(gate_up[r, c], gate_up[r, inter + c]).  "silu": silu(g) * u.  "capped_swish":
-    g <- min(g, limit), u <- clamp(u, -limit, limit), g * sigmoid(alpha * g) * (u + 1)."""
+    g <- min(g, limit), u <- clamp(u, -limit, limit), g * sigmoid(alpha * g) * (u + 1).  "gelu_tanh": gelu(g) * u in
+    gelu's tanh form."""
     if activation == "silu":
         return silu_mul(gate_up, out)
     _need_cuda(gate_up, out)
@@ -198,6 +207,25 @@ def add_rmsnorm(residual: torch.Tensor, delta: Optional[torch.Tensor], gain: tor
               _ptr(gain), _ptr(out), _dtype_code(out), _ptr(rows), n, d, float(eps), _stream()),
            "add_rmsnorm")
     return out
+
+
+def norm_add(x: torch.Tensor, y: torch.Tensor, gain: torch.Tensor, eps: float,
+             lp_dtype: Optional[torch.dtype] = None) -> Optional[torch.Tensor]:
+    """x += gain * y / sqrt(mean(y^2) + eps), in place: x float32 [T, W], y [T, W] in float32 or bfloat16,
+    gain float32 [W].  Returns a copy of the new x in ``lp_dtype`` (y's dtype), or None when that is None."""
+    _need_cuda(x, y, gain)
+    _need_contiguous(x, y, gain)
+    if x.dtype != torch.float32 or x.dim() != 2 or y.shape != x.shape:
+        raise KernelError("norm_add: x is float32 [T, W] and y has its shape")
+    T, d = x.shape
+    if gain.dtype != torch.float32 or gain.numel() != d:
+        raise KernelError("norm_add: the gain is float32 [W]")
+    if lp_dtype is not None and lp_dtype != y.dtype:
+        raise KernelError("norm_add: the copy has y's dtype")
+    lp = torch.empty((T, d), dtype=lp_dtype, device=x.device) if lp_dtype is not None else None
+    fn = _fn("norm_add", "pbe_norm_add", [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p])
+    _check(fn(_ptr(x), _ptr(y), _dtype_code(y), _ptr(gain), _ptr(lp), T, d, float(eps), _stream()), "norm_add")
+    return lp
 
 
 def silu_mul(gate_up: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
@@ -282,16 +310,17 @@ def gated_rms(o: torch.Tensor, gate: torch.Tensor, gain: Optional[torch.Tensor],
     T, N = o.shape
     if o.dtype != torch.float32 or N % heads or tuple(gate.shape) != (T, N) or gate.stride(1) != 1:
         raise KernelError("gated_rms: shapes, strides or dtypes do not agree")
-    if gate.dtype != out_dtype:
-        raise KernelError("gated_rms: the gate has the output's dtype")
+    if gate.dtype not in (out_dtype, torch.float32):
+        raise KernelError("gated_rms: the gate has the output's dtype or is float32")
     if gain is not None and (gain.dtype != torch.float32 or gain.numel() != N):
         raise KernelError("gated_rms: gain must be float32 [heads * E]")
     if gate_act not in ("sigmoid", "silu"):
         raise KernelError(f"gated_rms: unknown gate activation {gate_act!r}")
     out = torch.empty((T, N), dtype=out_dtype, device=o.device)
-    fn = _fn("streams", "pbe_gated_rms", [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
-                                          c_float, c_int, c_int, c_int, c_void_p])
-    _check(fn(_ptr(o), _ptr(gate), gate.stride(0) if T > 1 else N, _ptr(gain), _ptr(out), _dtype_code(out), T, heads,
+    fn = _fn("streams", "pbe_gated_rms", [c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
+                                          c_int, c_float, c_int, c_int, c_int, c_void_p])
+    _check(fn(_ptr(o), _ptr(gate), _dtype_code(gate), gate.stride(0) if T > 1 else N, _ptr(gain), _ptr(out),
+              _dtype_code(out), T, heads,
               N // heads, float(eps), 1 if per_head else 0, 1 if gate_act == "silu" else 0, 1 if gate_first else 0,
               _stream()), "gated_rms")
     return out
@@ -581,9 +610,11 @@ SKINNY_MAX_ROWS = int(os.environ.get('PBE_SKINNY_ROWS', '8'))      # batches of 
 
 
 def gemm_skinny(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
-                out_dtype: Optional[torch.dtype] = None, swiglu: bool = False) -> torch.Tensor:
+                out_dtype: Optional[torch.dtype] = None, swiglu: bool = False,
+                activation: str = "silu") -> torch.Tensor:
     """y = x w^T (+ b) for at most 16 rows, bfloat16 operands, weights streamed once.
-    ``swiglu``: w is [gate; up] stacked and y = silu(x gate^T) * (x up^T), [M, N/2]."""
+    ``swiglu``: w is [gate; up] stacked and y = act(x gate^T) * (x up^T), [M, N/2], with ``activation``
+    one of ``GLU_EPILOGUES``."""
     _need_cuda(x, w, bias)
     _need_contiguous(x, w, bias)
     M, K = x.shape
@@ -600,8 +631,8 @@ def gemm_skinny(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] =
     out = torch.empty((M, N // 2 if swiglu else N), dtype=out_dtype, device=x.device)
     fn = _fn("gemm_skinny", "pbe_gemm_skinny",
              [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p])
-    _check(fn(_ptr(x), _ptr(w), _ptr(bias), _ptr(out), _dtype_code(out), M, N, K, 1 if swiglu else 0,
-              _stream()), "gemm_skinny")
+    _check(fn(_ptr(x), _ptr(w), _ptr(bias), _ptr(out), _dtype_code(out), M, N, K,
+              GLU_EPILOGUES[activation] if swiglu else 0, _stream()), "gemm_skinny")
     return out
 
 
@@ -648,11 +679,11 @@ _stream_state = {}     # per device: (scratch floats, zeroed tickets) of the K-s
 
 
 def gemm_stream(x: torch.Tensor, w: torch.Tensor, out_dtype: Optional[torch.dtype] = None,
-                swiglu: bool = False, check: bool = False) -> torch.Tensor:
+                swiglu: bool = False, check: bool = False, activation: str = "silu") -> torch.Tensor:
     """y = x w^T for up to 64 rows on the tcgen05 tensor cores with the weights as the streamed
     operand (TMA-fed ring, accumulator in tensor memory, K split over blocks where the matrix has
-    few rows).  ``swiglu``: w is [gate; up] stacked and y = silu(x gate^T) * (x up^T), [M, N/2].
-    ``check`` synchronises and raises if a bounded wait inside the kernel ran out."""
+    few rows).  ``swiglu``: w is [gate; up] stacked and y = act(x gate^T) * (x up^T), [M, N/2], with
+    ``activation`` one of ``GLU_EPILOGUES``.  ``check`` synchronises and raises if a bounded wait inside the kernel ran out."""
     _need_cuda(x, w)
     _need_contiguous(x, w)
     M, K = x.shape
@@ -668,8 +699,8 @@ def gemm_stream(x: torch.Tensor, w: torch.Tensor, out_dtype: Optional[torch.dtyp
     scratch, tickets, err = gemm_stream_buffers(x.device)
     fn = _fn("gemm_stream", "pbe_gemm_stream",
              [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p])
-    _check(fn(_ptr(x), _ptr(w), _ptr(out), _dtype_code(out), M, N, K, 1 if swiglu else 0, _ptr(scratch), _ptr(tickets),
-              _ptr(err), _stream()), "gemm_stream")
+    _check(fn(_ptr(x), _ptr(w), _ptr(out), _dtype_code(out), M, N, K, GLU_EPILOGUES[activation] if swiglu else 0,
+              _ptr(scratch), _ptr(tickets), _ptr(err), _stream()), "gemm_stream")
     if check and int(err.item()) != 0:
         err.zero_()
         raise KernelError("gemm_stream: a wait inside the kernel ran out; the result is invalid")
@@ -1460,16 +1491,32 @@ def head_norm_write(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, bias
                     q_gain: Optional[torch.Tensor], k_gain: Optional[torch.Tensor], slots: Optional[torch.Tensor],
                     k_pages: Optional[torch.Tensor], v_pages: Optional[torch.Tensor], num_heads: int,
                     num_kv_heads: int, key_dim: int, value_dim: int, page_tokens: int, eps: float,
-                    q_head_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
+                    q_head_scale: Optional[torch.Tensor] = None, positions: Optional[torch.Tensor] = None,
+                    rot_freq: Optional[torch.Tensor] = None, value_freq: Optional[torch.Tensor] = None):
     """From a fused projection [T, ld] (queries at column ``q_off``, keys at ``k_off``, values at
     ``v_off``): ``bias`` (float32, indexed like the columns) added, an RMS norm over each query and
     key head's ``key_dim`` elements with the gains ``q_gain`` / ``k_gain`` (float32 [key_dim], shared
     by the heads; None: no norm), all in float32; ``q_head_scale`` (float32 [H]) multiplies head h's
     normed query (a temperature per head).  Returns the queries, float32 [T, H * D]; keys go to
     ``k_pages`` [page, G, page_tokens, D] and values to ``v_pages`` [page, G, page_tokens, E] at
-    ``slots`` (None or a negative slot: nothing is written)."""
-    _need_cuda(proj, bias, q_gain, k_gain, slots, k_pages, v_pages, q_head_scale)
-    _need_contiguous(bias, q_gain, k_gain, slots, k_pages, v_pages, q_head_scale)
+    ``slots`` (None or a negative slot: nothing is written).
+
+    Rotations by the row's position (``positions`` int32 [T]), halves paired, frequencies from
+    ``turn_frequencies``: ``rot_freq`` [n, 2] turns the first 2n dimensions of every normed query and
+    key, ``value_freq`` [E / 2, 2] turns whole values.  With ``value_freq`` the result is (queries,
+    table), the table float32 [T, E / 2, 2] of the values' (cos, sin) that ``masked_attention`` turns
+    its outputs back by."""
+    _need_cuda(proj, bias, q_gain, k_gain, slots, k_pages, v_pages, q_head_scale, positions, rot_freq, value_freq)
+    _need_contiguous(bias, q_gain, k_gain, slots, k_pages, v_pages, q_head_scale, positions, rot_freq, value_freq)
+    if rot_freq is not None or value_freq is not None:
+        if positions is None or positions.dtype != torch.int32 or positions.numel() != proj.shape[0]:
+            raise KernelError("head_norm_write: a rotation needs the rows' positions, int32 [T]")
+    for name, f, width in (("rot_freq", rot_freq, key_dim), ("value_freq", value_freq, value_dim)):
+        if f is not None and (f.dtype != torch.float32 or f.dim() != 2 or f.shape[1] != 2 or 2 * f.shape[0] > width
+                              or f.shape[0] < 1):
+            raise KernelError(f"head_norm_write: {name} is float32 [pairs, 2] and its pairs fit into a head")
+    if value_freq is not None and (2 * value_freq.shape[0] != value_dim or value_dim > 256):
+        raise KernelError("head_norm_write: whole values turn; they are even and at most 256 wide")
     if q_head_scale is not None and (q_head_scale.dtype != torch.float32 or q_head_scale.numel() != num_heads):
         raise KernelError("head_norm_write: the heads' factors are float32 [H]")
     if proj.dim() != 2 or proj.stride(1) != 1:
@@ -1488,32 +1535,54 @@ def head_norm_write(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, bias
                                 or v_pages is None or tuple(v_pages.shape[1:]) != (G, page_tokens, E)):
         raise KernelError("head_norm_write: pages are [page, G, page_tokens, D] and [page, G, page_tokens, E]")
     q = torch.empty((T, H * D), dtype=torch.float32, device=proj.device)
+    turn = None
+    if value_freq is not None:
+        turn = torch.empty((T, E // 2, 2), dtype=torch.float32, device=proj.device)
     fn = _fn("masked_attention", "pbe_head_norm_write",
              [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-              c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p])
+              c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
+              c_int, c_void_p])
     _check(fn(_ptr(proj), proj.stride(0), int(q_off), int(k_off), int(v_off), _ptr(bias), _ptr(q_gain), _ptr(k_gain),
               _ptr(q_head_scale), _ptr(slots if k_pages is not None else None), _ptr(q), _ptr(k_pages), _ptr(v_pages), T, H, G, D, E,
-              int(page_tokens), float(eps), _dtype_code(proj), _stream()), "head_norm_write")
-    return q
+              int(page_tokens), float(eps), _ptr(positions), _ptr(rot_freq),
+              2 * rot_freq.shape[0] if rot_freq is not None else 0, _ptr(value_freq), _ptr(turn), _dtype_code(proj),
+              _stream()), "head_norm_write")
+    return q if turn is None else (q, turn)
+
+
+def turn_frequencies(pairs: int, base: float, device) -> torch.Tensor:
+    """base^(-i / pairs) for i = 0 .. pairs - 1 in turns a position (divided by 2 pi), float32 [pairs, 2]:
+    the rounded number and what the rounding left."""
+    i = torch.arange(pairs, dtype=torch.float64)
+    f = torch.pow(torch.tensor(float(base), dtype=torch.float64), -i / pairs) / (2.0 * math.pi)
+    hi = f.to(torch.float32)
+    return torch.stack([hi, (f - hi.double()).to(torch.float32)], dim=1).contiguous().to(device)
 
 
 def masked_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, meta, num_heads: int,
                      num_kv_heads: int, scale: float, mask: Optional[str], mask_size: Optional[int],
                      page_tokens: int, bias: Optional[torch.Tensor] = None, unit_sink: bool = False,
-                     gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     gate: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None,
+                     softcap: Optional[float] = None, turn: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Softmax attention of every row over its request's pages.  ``q`` float32 [T, H * D]; pages
     [page, G, page_tokens, D] and [page, G, page_tokens, E].  ``mask``: None / "causal" (every earlier
     key), "window" (the last ``mask_size`` keys) or "chunk" (the earlier keys of the row's own chunk of
     ``mask_size`` positions).  ``bias`` float32 [H, rows]: bias[h, min(distance, rows - 1)] is added to
-    the scaled score.  ``unit_sink``: one more term e^0 in the denominator.  ``gate`` [T, >= H * E] (a
-    column slice in the pages' dtype): the output times its sigmoid.  ``meta``: the step's work list
+    the scaled score.  ``softcap`` c: the scaled score becomes c * tanh(score / c) (before the bias).
+    ``unit_sink``: one more term e^0 in the denominator; ``sink`` float32 [H]: one more term e^sink[h].
+    ``turn`` (from ``head_norm_write``): every head's output is turned back by its row's angles, before
+    the gate.  ``gate`` [T, >= H * E] (a column slice in the pages' dtype): the output times its sigmoid.  ``meta``: the step's work list
     for (group, H / G, ``masked_tile_rows(dtype, D, E)``, ``mask_size``).  Returns [T, H * E] in the
     pages' dtype.  Arithmetic is float32 throughout; on the tensor-core path the float32 queries and
     softmax weights enter the products as two bfloat16 numbers each."""
-    _need_cuda(q, k_pages, v_pages, bias, gate)
-    _need_contiguous(q, k_pages, v_pages, bias)
+    _need_cuda(q, k_pages, v_pages, bias, gate, sink, turn)
+    _need_contiguous(q, k_pages, v_pages, bias, sink, turn)
     T = q.shape[0]
     H, G = num_heads, num_kv_heads
+    if sink is not None and (sink.dtype != torch.float32 or sink.numel() != H or unit_sink):
+        raise KernelError("masked_attention: the sink is float32 [H], and there is one sink only")
+    if softcap is not None and not softcap > 0:
+        raise KernelError("masked_attention: a cap is positive")
     D, E = k_pages.shape[-1], v_pages.shape[-1]
     if q.dtype != torch.float32 or q.shape[1] != H * D or k_pages.dtype != v_pages.dtype:
         raise KernelError("masked_attention: q is float32 [T, H * D]; the pages share a dtype")
@@ -1525,6 +1594,9 @@ def masked_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tens
         raise KernelError("masked_attention: the gate is a column slice [T, H * E] in the pages' dtype")
     if E > 256:
         raise KernelError("masked_attention: values are at most 256 wide")
+    if turn is not None and (turn.dtype != torch.float32 or tuple(turn.shape) != (T, E // 2, 2) or E % 2):
+        raise KernelError("masked_attention: the table of turns is float32 [T, E / 2, 2]")
+    has_sink = 1 if (unit_sink or sink is not None) else 0
     out = torch.empty((T, H * E), dtype=k_pages.dtype, device=q.device)
     part_o = part_ml = None
     if meta.num_split_rows:
@@ -1547,24 +1619,26 @@ def masked_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tens
         tile_rows=int(meta.tile_rows), scale=float(scale), kinds=0, num_pages=int(k_pages.shape[0]))
     if masked_mma_applies(k_pages.dtype, D, E):
         fn = _fn("masked_attention_mma", "pbe_masked_attention_mma",
-                 [ctypes.POINTER(AttnParams), c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p],
+                 [ctypes.POINTER(AttnParams), c_void_p, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_void_p, c_int,
+                  c_int, c_void_p],
                  {"PBE_MA_D": int(D), "PBE_MA_E": int(E)})
         _check(fn(ctypes.byref(p), _ptr(bias), bias.shape[1] if bias is not None else 0, MASK_KINDS[mask],
-                  1 if unit_sink else 0, _ptr(gate), int(ldg), int(meta.num_work), _stream()), "masked_attention_mma")
+                  has_sink, _ptr(sink), float(softcap or 0.0), _ptr(turn), _ptr(gate), int(ldg), int(meta.num_work),
+                  _stream()), "masked_attention_mma")
     else:
         fn = _fn("masked_attention", "pbe_masked_attention",
-                 [ctypes.POINTER(AttnParams), c_int, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int,
-                  c_int, c_void_p])
+                 [ctypes.POINTER(AttnParams), c_int, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_float, c_void_p,
+                  c_void_p, c_int, c_int, c_int, c_void_p])
         _check(fn(ctypes.byref(p), int(D), int(E), _ptr(bias), bias.shape[1] if bias is not None else 0,
-                  MASK_KINDS[mask], 1 if unit_sink else 0, _ptr(gate), int(ldg), int(meta.num_work),
-                  _dtype_code(k_pages), _stream()), "masked_attention")
+                  MASK_KINDS[mask], has_sink, _ptr(sink), float(softcap or 0.0), _ptr(turn), _ptr(gate), int(ldg),
+                  int(meta.num_work), _dtype_code(k_pages), _stream()), "masked_attention")
     if meta.num_split_rows > 0:
         mp = AttnMergeParams(part_o=part_o.data_ptr(), part_ml=part_ml.data_ptr(), out=out.data_ptr(),
                              split_tokens=meta.split_tokens.data_ptr(), split_counts=meta.split_counts.data_ptr(),
                              num_heads=int(H), head_dim=int(E), max_splits=int(meta.max_splits))
         mfn = _fn("masked_attention", "pbe_masked_merge",
-                  [ctypes.POINTER(AttnMergeParams), c_int, c_void_p, c_int, c_int, c_int, c_void_p])
-        _check(mfn(ctypes.byref(mp), 1 if unit_sink else 0, _ptr(gate), int(ldg), int(meta.num_split_rows),
+                  [ctypes.POINTER(AttnMergeParams), c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p])
+        _check(mfn(ctypes.byref(mp), has_sink, _ptr(sink), _ptr(turn), _ptr(gate), int(ldg), int(meta.num_split_rows),
                    _dtype_code(k_pages), _stream()), "masked_merge")
     return out
 
@@ -1926,4 +2000,94 @@ def gated_scan(a: Optional[torch.Tensor], b: Optional[torch.Tensor], y: Optional
            "chunk_starts")
     _check(fn(*coeff, _ptr(y), ldy, _ptr(out), code, _ptr(state), _ptr(scratch_s), _ptr(scratch_p),
               _ptr(plan.second_pass), plan.num_second_pass, None, None, None, C, act, 2, _stream()), "gated_scan")
+    return out
+
+
+# ------------------------------------------------------------------ gated delta rule
+def delta_inputs(proj: torch.Tensor, conv_t: torch.Tensor, conv_state: torch.Tensor, small: torch.Tensor,
+                 chan: Optional[torch.Tensor], dt_bias: torch.Tensor, a_log: torch.Tensor, request_of_row: torch.Tensor,
+                 q_start: torch.Tensor, q_len: torch.Tensor, slots: torch.Tensor, num_requests: int, kv_heads: int,
+                 heads: int, dim: int, vdim: int, q_scale: float, unit_eps: float, update_state: bool = True,
+                 single_tokens: bool = False):
+    """Everything that enters a gated delta rule, float32, from a projection [T, ld] whose columns begin
+    with q [G * D], k [G * D], v [H * E]: the causal convolutions (``conv_t`` float32 [taps, C], the last
+    tap on the current token; ``conv_state`` float32 [slots, taps - 1, C], read and moved on) and silu;
+    q and k as unit vectors x / sqrt(sum(x^2) + unit_eps), q times ``q_scale``; beta = sigmoid of
+    ``small`` [T, :H] (float32); decays exp(-exp(a_log_h) softplus(x + dt_bias)) with x = ``small``
+    [T, H:2H] (one per head) or ``chan`` [T, H * D] (float32; one per head and key channel).
+    ``single_tokens``: every request of the step brings one token.
+    Returns (qk [T, G, 2, D], k . q [T, G], v [T, H * E], beta [T, H], decay [T, H] or [T, H * D])."""
+    _need_cuda(proj, conv_t, conv_state, small, chan, dt_bias, a_log, request_of_row, q_start, q_len, slots)
+    _need_contiguous(conv_t, conv_state, dt_bias, a_log)
+    G, H, D, E = kv_heads, heads, dim, vdim
+    C = 2 * G * D + H * E
+    taps = conv_t.shape[0]
+    T = proj.shape[0]
+    if proj.dim() != 2 or proj.stride(1) != 1 or proj.shape[1] < C or H % G:
+        raise KernelError("delta_inputs: the projection is [T, >= 2 G D + H E] with unit column stride")
+    if D > 512 or E > 512 or not 1 <= taps <= 16:
+        raise KernelError("delta_inputs: heads are at most 512 wide, and there are 1 to 16 taps")
+    if conv_t.dtype != torch.float32 or conv_t.shape[1] != C or conv_state.dtype != torch.float32 or \
+            tuple(conv_state.shape[1:]) != (taps - 1, C):
+        raise KernelError("delta_inputs: conv_t is float32 [taps, C], the state float32 [slots, taps - 1, C]")
+    n_small, n_dt = (H, H * D) if chan is not None else (2 * H, H)
+    for name, x, n in (("small", small, n_small), ("chan", chan, H * D)):
+        if x is not None and (x.dtype != torch.float32 or x.dim() != 2 or x.shape[0] != T or x.shape[1] < n
+                              or x.stride(1) != 1):
+            raise KernelError(f"delta_inputs: {name} is float32 [T, >= {n}] with unit column stride")
+    if dt_bias.dtype != torch.float32 or dt_bias.numel() != n_dt or a_log.dtype != torch.float32 or a_log.numel() != H:
+        raise KernelError("delta_inputs: dt_bias has a number per decay and a_log one per head, float32")
+    for x in (request_of_row, q_start, q_len, slots):
+        if x.dtype != torch.int32:
+            raise KernelError("delta_inputs: the step's arrays are int32")
+    dev = proj.device
+    qk = torch.empty((T, G, 2, D), dtype=torch.float32, device=dev)
+    kq = torch.empty((T, G), dtype=torch.float32, device=dev)
+    v = torch.empty((T, H * E), dtype=torch.float32, device=dev)
+    beta = torch.empty((T, H), dtype=torch.float32, device=dev)
+    decay = torch.empty((T, n_dt), dtype=torch.float32, device=dev)
+
+    def ld(x):
+        return 0 if x is None else (x.stride(0) if T > 1 else max(x.stride(0), x.shape[1]))
+    many = not single_tokens
+    fn = _fn("delta_rule", "pbe_delta_inputs",
+             [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int] + [c_void_p] * 11
+             + [c_int] * 9 + [c_float, c_float, c_void_p])
+    global _launches
+    _check(fn(_ptr(proj), ld(proj), _dtype_code(proj), _ptr(conv_t), _ptr(conv_state), _ptr(small), ld(small), _ptr(chan),
+              ld(chan), _ptr(dt_bias), _ptr(a_log), _ptr(qk), _ptr(kq), _ptr(v), _ptr(beta), _ptr(decay),
+              _ptr(request_of_row), _ptr(q_start), _ptr(q_len), _ptr(slots), T, int(num_requests), G, H, D, E, taps,
+              1 if update_state else 0, 1 if many else 0, float(q_scale), float(unit_eps), _stream()), "delta_inputs")
+    if many and update_state and taps > 1:
+        _launches += 1
+    return qk, kq, v, beta, decay
+
+
+def delta_scan(qk: torch.Tensor, kq: torch.Tensor, v: torch.Tensor, beta: torch.Tensor, decay: torch.Tensor,
+               state: torch.Tensor, q_start: torch.Tensor, q_len: torch.Tensor, slots: torch.Tensor, num_requests: int,
+               update_state: bool = True, zero_out: bool = False) -> torch.Tensor:
+    """The gated delta rule request by request over the rows each brings: S <- g S,
+    u = beta (v - S^T k), S <- S + k u^T, o = S^T q, with the inputs of ``delta_inputs`` and ``state``
+    float32 [slots, H, E, D] (S transposed: a value column's key channels side by side), read at
+    ``slots[r]`` and left updated.  Returns o, float32 [T, H * E]."""
+    _need_cuda(qk, kq, v, beta, decay, state, q_start, q_len, slots)
+    _need_contiguous(qk, kq, v, beta, decay, state)
+    T, G, _, D = qk.shape
+    H = beta.shape[1]
+    E = v.shape[1] // H
+    for x in (qk, kq, v, beta, decay, state):
+        if x.dtype != torch.float32:
+            raise KernelError("delta_scan: everything is float32")
+    if H % G or tuple(kq.shape) != (T, G) or v.shape[0] != T or v.shape[1] != H * E or beta.shape[0] != T or \
+            decay.shape[0] != T or decay.shape[1] not in (H, H * D) or tuple(state.shape[1:]) != (H, E, D):
+        raise KernelError("delta_scan: shapes do not agree")
+    for x in (q_start, q_len, slots):
+        if x.dtype != torch.int32 or x.numel() < num_requests:
+            raise KernelError("delta_scan: request arrays are int32 [R]")
+    per_channel = decay.shape[1] == H * D and D > 1
+    out = (torch.zeros if zero_out else torch.empty)((T, H * E), dtype=torch.float32, device=v.device)
+    fn = _fn("delta_rule", "pbe_delta_scan", [c_void_p] * 5 + [c_int] + [c_void_p] * 5 + [c_int] * 6 + [c_void_p])
+    _check(fn(_ptr(qk), _ptr(kq), _ptr(v), _ptr(beta), _ptr(decay), 1 if per_channel else 0, _ptr(out), _ptr(state),
+              _ptr(q_start), _ptr(q_len), _ptr(slots), int(num_requests), G, H, D, E, 1 if update_state else 0,
+              _stream()), "delta_scan")
     return out

@@ -32,10 +32,9 @@ class DecoderModel:
                 raise TypeError("the embedding's norm must be able to norm gathered rows (ScalarRMSNorm)")
         if spec.depth_stack not in (None, "mix", "plain"):
             raise ValueError(f"unknown depth_stack {spec.depth_stack!r}")
-        if spec.depth_stack is not None and (spec.residual_streams != 1 or spec.embedding_scale != 1.0
-                                             or spec.position_table_name is not None
+        if spec.depth_stack is not None and (spec.residual_streams != 1
                                              or any(st.input_mix for st in spec.run_order)):
-            raise ValueError("a depth stack goes with one residual stream, an unscaled embedding and no input mixes")
+            raise ValueError("a depth stack goes with one residual stream and no input mixes")
         self.embed = None
         self.lm_head = None
         self.position_table = None
@@ -194,8 +193,9 @@ class DecoderModel:
                                                  stack.lp_dtype() if stack is not None else None)
         elif s.embedding_scale != 1.0 or self.position_table is not None:
             # a learned position row follows the token's place in the sequence
-            ops.embedding_positions(residual, self.embed, ctx.token_ids, s.embedding_scale, self.position_table,
-                                    ctx.positions)
+            first_lp = ops.embedding_positions(residual, self.embed, ctx.token_ids, s.embedding_scale,
+                                               self.position_table, ctx.positions,
+                                               stack.lp_dtype() if stack is not None else None)
         else:
             ops.embedding(residual, self.embed, ctx.token_ids)
         first = None

@@ -5,8 +5,9 @@ from .rope import NoPositionEncoding, RotaryEncoding
 from .attention import GQAttention
 from .mlp import ActivationMLP, SwiGLU
 from .routed_experts import RoutedExperts
-from .block import DepthStack, ParallelBlock, PostNormBlock, PreNormBlock
+from .block import DepthStack, OutputNormBlock, ParallelBlock, PostNormBlock, PreNormBlock
 from .gated_recurrence import GatedLinearRecurrence
+from .delta_rule import GatedDeltaRule
 from .linear_attention import DecayLinearAttention
 from .pooled_attention import PooledWindowAttention
 from .parallel import ParallelMixer
@@ -21,4 +22,5 @@ __all__ = ["Block", "CacheTensor", "CompositeNeed", "FeedForward", "KVNeed", "Mi
            "GQAttention", "SwiGLU", "PreNormBlock", "LayerNorm", "PendingUpdate", "DecayLinearAttention",
            "PooledWindowAttention", "ParallelMixer", "StreamBlock", "StreamConnection", "DeltaSum", "ActivationMLP",
            "RoutedExperts", "ParallelBlock", "SelectiveStateSpace", "LatentAttention", "MaskedAttention",
-           "ScalarRMSNorm", "DepthStack", "PostNormBlock", "GatedLinearRecurrence"]
+           "ScalarRMSNorm", "DepthStack", "PostNormBlock", "GatedLinearRecurrence",
+           "OutputNormBlock", "GatedDeltaRule"]

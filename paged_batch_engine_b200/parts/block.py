@@ -138,6 +138,10 @@ class DepthStack:
     def next_mixed(self):
         return self.mixed[self.filled & 1] if self.mixes else None
 
+    def update(self, lp):
+        """``current`` was changed in place; ``lp`` is its new rounding (None in float32 runs)."""
+        self.current_lp = lp if lp is not None else self.current
+
     def push(self, mixed, lp):
         """The layer run's result is in ``next_result()`` (and its mix over depth in ``mixed``)."""
         result = self.next_result()
@@ -228,6 +232,57 @@ class PostNormBlock(Block):
         return st, None
 
 
+class OutputNormBlock(Block):
+    """Norm on what a sublayer returns: x <- x + n1(mixer(x)), then (with a feed-forward) x <- x +
+    n2(feed_forward(x)); the sublayers read the stream itself.  The residual is a ``DepthStack`` whose
+    current stream is updated in place: the norm's launch forms n(y), adds it to the float32 stream and
+    leaves the sum's rounding to the run dtype beside it, which the next product reads."""
+
+    def __init__(self, spec: BlockSpec, dtype, device):
+        self.spec = spec
+        self.prefix = spec.prefix
+        n = spec.names
+        self.p_mixer = self.prefix + n.get("mixer", "mixer.")
+        self.p_ffn = self.prefix + n.get("feed_forward", "feed_forward.")
+        self.p_norm1 = self.prefix + n.get("norm_mixer", "norm_mixer.")
+        self.p_norm2 = self.prefix + n.get("norm_feed_forward", "norm_feed_forward.")
+        self.norm1 = build_part("norm", spec.norm_mixer, dtype, device)
+        self.mixer = build_part("mixer", spec.mixer, dtype, device)
+        self.norm2 = self.ffn = None
+        if spec.feed_forward is not None:
+            self.norm2 = build_part("norm", spec.norm_feed_forward, dtype, device)
+            self.ffn = build_part("feed_forward", spec.feed_forward, dtype, device)
+        for norm in (self.norm1, self.norm2):
+            if norm is not None and not (hasattr(norm, "norm_add") and norm.on_output):
+                raise TypeError("an output-norm block needs norms that add to the stream (RMSNorm with on_output)")
+
+    def parts(self):
+        out = [(self.norm1, self.p_norm1), (self.mixer, self.p_mixer)]
+        if self.ffn is not None:
+            out += [(self.norm2, self.p_norm2), (self.ffn, self.p_ffn)]
+        return out
+
+    def param_specs(self, prefix=""):
+        return [s for part, p in self.parts() for s in part.param_specs(p)]
+
+    def load(self, tensors, prefix=""):
+        for part, p in self.parts():
+            part.load(tensors, p)
+
+    def kernel_libraries(self, dtype):
+        return [lib for part, _ in self.parts() for lib in part.kernel_libraries(dtype)]
+
+    def forward(self, residual, delta, ctx, cache):
+        if not isinstance(residual, DepthStack) or residual.mixes or delta is not None:
+            raise TypeError('output-norm blocks pass a DepthStack along ("plain") and leave nothing pending')
+        st = residual
+        st.update(self.norm1.norm_add(st.current, self.mixer.forward(st.current_lp, ctx, cache), st.lp_dtype()))
+        if self.ffn is not None:
+            st.update(self.norm2.norm_add(st.current, self.ffn.forward(st.current_lp, ctx), st.lp_dtype()))
+        return st, None
+
+
+register_part("block", "outnorm", lambda spec, dtype, device: OutputNormBlock(spec, dtype, device), replace=True)
 register_part("block", "postnorm", lambda spec, dtype, device: PostNormBlock(spec, dtype, device), replace=True)
 register_part("block", "prenorm", lambda spec, dtype, device: PreNormBlock(spec, dtype, device),
               replace=True)

@@ -1,5 +1,5 @@
-"""Grouped-query softmax attention with per-head query/key norms and a choice of mask, score
-bias, sink and gate."""
+"""Grouped-query softmax attention with per-head query/key norms, optional rotations of queries, keys
+and values, and a choice of mask, score cap, score bias, sink and gate."""
 from __future__ import annotations
 
 import math
@@ -26,7 +26,7 @@ def log_bucket(distance: int, rows: int, far: float) -> int:
 class MaskedAttention(Mixer):
     """q, k, v (and the gate) = x W^T as one fused product; an RMS norm over each query and key
     head with one gain vector per projection, shared by the heads (``qk_norm``; "unit": the heads
-    are divided by their root mean square and there are no gain tensors); no rotation;
+    are divided by their root mean square and there are no gain tensors); ``rotary`` or no rotation;
     score = q . k * ``scale`` (times a learned number per query head, ``head_temperature``: tensor
     ``temp`` [H]) (+ a learned bias by head and distance bucket, ``distance_bias``);
     softmax over the keys the mask lets the row see; output projection.
@@ -39,6 +39,13 @@ class MaskedAttention(Mixer):
     rel[bucket(i - j), h] with ``log_bucket``; the scale does not multiply it.  B is the checkpoint
     tensor's own first size (``rows`` only says how many to make when weights are drawn at random).
     ``unit_sink``: the softmax's denominator has one more term e^0 that carries no value.
+    ``sink``: the same with e^s, s a learned number per head (tensor ``sink`` [H]; neither scaled nor capped).
+    ``softcap`` c: the scaled score becomes c tanh(score / c) before the bias is added.
+    ``rotary`` dict(dims=n, base=b): after the norm the first n dimensions of every query and key turn by
+    the token's position, dimension i with i + n/2 by position * b^(-2i/n) (halves paired); keys are
+    cached so.  ``rotate_values``: the value of position j turns by j over all ``value_dim`` dimensions in
+    the same way (base ``rotary["base"]``) and is cached so; each head's output at position i turns back
+    by i, ahead of the gate.
     ``out_gate``: the concatenated heads are multiplied by sigmoid(W_g x) element by element.
     ``proj_bias``: q, k, v and the output projection have biases (``<name>.b``); "qkv": only q, k and v.
     Keys are ``key_dim`` wide and values ``value_dim``.
@@ -47,17 +54,18 @@ class MaskedAttention(Mixer):
     them are given back (a chunk is a subset of the window of its size).
 
     Checkpoint tensors under the prefix: q [H*D, hidden], k [G*D, hidden], v [G*E, hidden], o
-    [hidden, H*E], q.norm / k.norm [D], rel [B, H], g [H*E, hidden], and ``.b`` beside q, k, v, o
+    [hidden, H*E], q.norm / k.norm [D], rel [B, H], sink [H], g [H*E, hidden], and ``.b`` beside q, k, v, o
     (``tensor_names`` renames them)."""
     TENSOR_NAMES = dict(q="q", k="k", v="v", o="o", q_norm="q.norm", k_norm="k.norm", rel="rel", g="g",
-                        temp="temp", bias_suffix=".b")
+                        temp="temp", sink="sink", bias_suffix=".b")
     decode_capturable = True      # stepped from the step's device arrays alone
 
     def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, key_dim: int, value_dim: int,
                  scale: float, eps: float, dtype, device, mask: Optional[str] = None,
                  mask_size: Optional[int] = None, qk_norm: bool = True, distance_bias: Optional[dict] = None,
                  unit_sink: bool = False, out_gate: bool = False, proj_bias=False,
-                 head_temperature: bool = False, tensor_names: Optional[dict] = None):
+                 head_temperature: bool = False, sink: bool = False, softcap: Optional[float] = None,
+                 rotary: Optional[dict] = None, rotate_values: bool = False, tensor_names: Optional[dict] = None):
         unknown = set(tensor_names or {}) - set(self.TENSOR_NAMES)
         if unknown:
             raise ValueError(f"tensor_names knows {sorted(self.TENSOR_NAMES)}; got {sorted(unknown)}")
@@ -85,7 +93,20 @@ class MaskedAttention(Mixer):
             self.bias_rows, self.bias_far = int(distance_bias.get("rows") or 16), float(distance_bias["far"])
             if mask != "window":
                 raise ValueError("a distance bias is tabulated over a window's distances")
+        self.sink, self.softcap = bool(sink), (float(softcap) if softcap is not None else None)
+        if self.sink and self.unit_sink:
+            raise ValueError("a softmax has one sink: the unit sink or a learned one")
+        if self.softcap is not None and not self.softcap > 0:
+            raise ValueError("softcap must be positive")
+        self.rot_dims = int(rotary["dims"]) if rotary else 0
+        self.rot_base = float(rotary["base"]) if rotary else None
+        self.rotate_values = bool(rotate_values)
+        if rotary and (self.rot_dims < 2 or self.rot_dims % 2 or self.rot_dims > key_dim):
+            raise ValueError("rotary dims are even, at least 2 and at most the key width")
+        if self.rotate_values and (not rotary or value_dim % 2):
+            raise ValueError("rotated values take the base of the rotation and an even width")
         self.dtype, self.device = dtype, device
+        self.rot_freq = self.value_freq = self.sink_scores = None
         self.tile_rows = ops.masked_tile_rows(dtype, key_dim, value_dim)
         self.w_in = self.b_in = self.w_o = self.b_o = self.q_gain = self.k_gain = self.bias_by_distance = None
         self.q_head_scale = None
@@ -125,6 +146,8 @@ class MaskedAttention(Mixer):
             specs.append(ParamSpec(prefix + n["temp"], (H,)))
         if self.bias_rows:
             specs.append(ParamSpec(prefix + n["rel"], (self.bias_rows, H), free_dims=(0,)))
+        if self.sink:
+            specs.append(ParamSpec(prefix + n["sink"], (H,)))
         if self.out_gate:
             specs.append(ParamSpec(prefix + n["g"], (H * E, w)))
         return specs
@@ -152,6 +175,12 @@ class MaskedAttention(Mixer):
             self.q_gain = self.k_gain = torch.ones(self.key_dim, dtype=torch.float32, device=self.w_in.device)
         if self.head_temperature:
             self.q_head_scale = tensors.pop(prefix + n["temp"]).to(torch.float32).contiguous()
+        if self.sink:
+            self.sink_scores = tensors.pop(prefix + n["sink"]).to(torch.float32).contiguous()
+        if self.rot_dims:
+            self.rot_freq = ops.turn_frequencies(self.rot_dims // 2, self.rot_base, self.w_in.device)
+        if self.rotate_values:
+            self.value_freq = ops.turn_frequencies(self.value_dim // 2, self.rot_base, self.w_in.device)
         if self.bias_rows:
             rel = tensors.pop(prefix + n["rel"]).to(torch.float32)
             self.bias_rows = int(rel.shape[0])
@@ -172,11 +201,14 @@ class MaskedAttention(Mixer):
         q = ops.head_norm_write(proj, q_off, k_off, v_off, self.b_in, self.q_gain, self.k_gain,
                                 group.slots if writes else None, cache.k if writes else None,
                                 cache.v if writes else None, H, G, D, E, ctx.page_tokens, self.eps,
-                                q_head_scale=self.q_head_scale)
+                                q_head_scale=self.q_head_scale, positions=ctx.position_ids if self.rot_dims else None,
+                                rot_freq=self.rot_freq, value_freq=self.value_freq)
+        q, turn = q if self.rotate_values else (q, None)
         meta = ctx.attention_work(cache.group, H // G, self.tile_rows, self.mask_size, H, E)
         gate = proj[:, g_off:] if self.out_gate else None
         out = ops.masked_attention(q, cache.k, cache.v, meta, H, G, self.scale, self.mask, self.mask_size,
-                                   ctx.page_tokens, bias=self.bias_by_distance, unit_sink=self.unit_sink, gate=gate)
+                                   ctx.page_tokens, bias=self.bias_by_distance, unit_sink=self.unit_sink, gate=gate,
+                                   sink=self.sink_scores, softcap=self.softcap, turn=turn)
         return ops.linear(out, self.w_o, self.b_o, out_dtype=self.dtype, kind=2)
 
 

@@ -9,15 +9,18 @@ from .base import FeedForward, register_part
 
 
 class SwiGLU(FeedForward):
-    """m = (silu(x W_gate^T) * (x W_up^T)) W_down^T, no biases; gate and up are one fused
-    product.  Reference: infMain/source/model/qwen2_batch.cpp:762-777 and
+    """m = (act(x W_gate^T) * (x W_up^T)) W_down^T, no biases; gate and up are one fused
+    product; ``activation`` "silu" or "gelu_tanh" (gelu's tanh form).  Reference: infMain/source/model/qwen2_batch.cpp:762-777 and
     swiglu_kernel.cu:6-25 (g * 1/(1+exp(-g)) * u in float32).
     Checkpoint tensors: gate_proj.weight, up_proj.weight [inter, hidden]; down_proj.weight
     [hidden, inter]; ``tensor_names`` renames them, e.g. ``dict(gate="w1", down="w2", up="w3")``."""
     TENSOR_NAMES = dict(gate="gate_proj", up="up_proj", down="down_proj")
 
     def __init__(self, hidden_size: int, intermediate_size: int, dtype, device, tensor_names=None,
-                 weight_suffix: str = ".weight"):
+                 weight_suffix: str = ".weight", activation: str = "silu"):
+        if activation not in ops.GLU_EPILOGUES:
+            raise ValueError(f"unknown activation {activation!r}; known: {', '.join(ops.GLU_EPILOGUES)}")
+        self.activation = activation
         self.suffix = weight_suffix      # what follows a projection's name in the checkpoint ("" for bare names)
         unknown = set(tensor_names or {}) - set(self.TENSOR_NAMES)
         if unknown:
@@ -49,17 +52,17 @@ class SwiGLU(FeedForward):
     def forward(self, x, ctx):
         # few rows (decode): the activation is the epilogue of a weight-streaming product
         if ops.stream_applies(x, self.w_gate_up, 4):
-            act = ops.gemm_stream(x, self.w_gate_up, self.dtype, swiglu=True)
+            act = ops.gemm_stream(x, self.w_gate_up, self.dtype, swiglu=True, activation=self.activation)
             return ops.linear(act, self.w_down, None, out_dtype=self.dtype, kind=8)
         if ops.skinny_applies(x, self.w_gate_up):
-            act = ops.gemm_skinny(x, self.w_gate_up, None, self.dtype, swiglu=True)
+            act = ops.gemm_skinny(x, self.w_gate_up, None, self.dtype, swiglu=True, activation=self.activation)
             return ops.linear(act, self.w_down, None, out_dtype=self.dtype, kind=8)
-        if ops.tc5_applies(x, self.w_gate_up, 4):
+        if self.activation == "silu" and ops.tc5_applies(x, self.w_gate_up, 4):
             act = ops.gemm_tc5(x, self.w_gate_up, self.dtype, swiglu=True)
             return ops.linear(act, self.w_down, None, out_dtype=self.dtype, kind=8)
         gu = ops.linear(x, self.w_gate_up, None, out_dtype=self.dtype, kind=32)
         act = torch.empty((x.shape[0], self.intermediate_size), dtype=self.dtype, device=x.device)
-        ops.silu_mul(gu, act)
+        ops.gated_activation(gu, act, self.activation)
         return ops.linear(act, self.w_down, None, out_dtype=self.dtype, kind=8)
 
 

@@ -18,15 +18,19 @@ class RMSNorm(Norm):
     one launch and the residual stream stays float32.
 
     ``one_plus``: the checkpoint stores the gain around zero, w = 1 + stored (formed once at load,
-    in float32)."""
+    in float32).  ``on_output``: the norm sits on a sublayer's output (``norm_add``)."""
 
-    def __init__(self, size: int, eps: float, dtype, device, weight_name: str = "weight", one_plus: bool = False):
+    def __init__(self, size: int, eps: float, dtype, device, weight_name: str = "weight", one_plus: bool = False,
+                 on_output: bool = False):
         self.size, self.eps, self.dtype, self.device = int(size), float(eps), dtype, device
-        self.weight_name, self.one_plus = weight_name, bool(one_plus)
+        self.weight_name, self.one_plus, self.on_output = weight_name, bool(one_plus), bool(on_output)
         self.gain = None
 
     def param_specs(self, prefix):
         return [ParamSpec(prefix + self.weight_name, (self.size,))]
+
+    def kernel_libraries(self, dtype):
+        return [("norm_add", None)] if self.on_output else []
 
     def load(self, tensors, prefix):
         self.gain = tensors[prefix + self.weight_name].to(torch.float32).contiguous()
@@ -40,6 +44,11 @@ class RMSNorm(Norm):
         n = residual.shape[0] if rows is None else rows.numel()
         out = torch.empty((n, self.size), dtype=out_dtype or self.dtype, device=residual.device)
         return ops.add_rmsnorm(residual, delta, self.gain, out, self.eps, rows)
+
+    def norm_add(self, x, y, lp_dtype):
+        """x += the norm of a sublayer's output ``y`` (x float32, in place); a copy of the new x in
+        ``lp_dtype`` is returned (None: no copy)."""
+        return ops.norm_add(x, y, self.gain, self.eps, lp_dtype)
 
     def add_norm_pair(self, other: "RMSNorm", residual, delta, out_dtype=None):
         """This norm and ``other`` of the same summed row (residual += delta first): the two differ
