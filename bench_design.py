@@ -1,13 +1,14 @@
 #!/usr/bin/env python3
 """A design beside the engine's closest existing model at equal layer sizes (random weights).
 
-    python bench.py --design gebadra|bavetar|gusorax|mobunex [--steps K] [--warmup W] [--sizes 2048,4096]
+    python bench.py --design gebadra|bavetar|gusorax|mobunex|tuterax [--steps K] [--warmup W] [--sizes 2048,4096]
 
 For each size: prefill (one 2,048-token prompt in one step) and decode (batch 8 from 2,048-token
 contexts, the captured decode step) throughput of a few layers of the design and of a Qwen2 model
 with the same width, heads, key/value heads, feed-forward width, vocabulary and number of
 layers (Mobunex stands beside Bavetar, the engine's closest model: latent attention, a recurrent
-layer behind a short convolution, routed experts); and the device time of the design's own kernels in one prompt step and one decode step,
+layer behind a short convolution, routed experts; Tuterax beside Mobunex - the same masked attention, a
+norm launch per sublayer - and Bavetar - a matrix state per head behind a short convolution); and the device time of the design's own kernels in one prompt step and one decode step,
 each beside the like kernel of the Qwen2 model, with the fraction of its roofline (the slower of
 algorithmic bytes over the measured copy bandwidth and algorithmic FLOPs over the measured bf16
 GEMM rate).  Times are CUDA events on the launching stream after warm-up; the per-kernel times
@@ -91,6 +92,22 @@ def mobunex_config(width: int) -> dict:
     layers = [dict(type="latent_attention", mixer=lat, mlp=dense), dict(type="attention", mixer=win, mlp=moe),
               dict(type="rglru", mixer=rec, mlp=moe), dict(type="latent_attention", mixer=lat, mlp=moe)][:LAYERS]
     return dict(architecture="Mobunex", width=width, vocab=32000, norm=dict(eps=1e-6), postln_alpha=1.5, layers=layers)
+
+
+def tuterax_config(width: int) -> dict:
+    """Four layers at the sizes of a real model of this kind: attention with heads of 128 (half of each
+    turned), an eighth as many key/value heads and a dense feed-forward, twice; between them a gated
+    delta rule with a decay per channel and one with a decay per head, as many heads as fill the width
+    with values of 128, half as many query/key heads of 128, 4 taps, no feed-forward."""
+    heads, ff = width // 128, {2048: 5632, 4096: 11008}.get(width, width * 11 // 4)
+    att = dict(heads=heads, kv_heads=max(1, heads // 8), dim=128, vdim=128, scale=128 ** -0.5, softcap=30.0,
+               rot=dict(base=1000000.0, dims=64))
+    delta = dict(heads=heads, kv_heads=max(1, heads // 2), dim=128, vdim=128, conv=4)
+    dense = dict(kind="dense", ff=ff)
+    layers = [dict(type="attention", mixer=att, mlp=dense), dict(type="channel_delta", mixer=delta, mlp=None),
+              dict(type="attention", mixer=att, mlp=dense), dict(type="delta", mixer=delta, mlp=None)][:LAYERS]
+    return dict(architecture="Tuterax", width=width, vocab=32000, norm=dict(eps=1e-6),
+                embedding=dict(scale=float(width) ** 0.5), layers=layers)
 
 
 def qwen_config(width: int, design: str = "gebadra") -> dict:
@@ -361,6 +378,44 @@ def rooflines_mobunex(width: int, pk: dict):
     return out
 
 
+def rooflines_tuterax(width: int, pk: dict):
+    """Algorithmic bytes and FLOPs of the compared kernels for the two workloads, per launch; the
+    recurrence's two kernels as the mean over the layer with a decay per channel and the one with a decay
+    per head."""
+    c = tuterax_config(width)
+    a, d = c["layers"][0]["mixer"], c["layers"][1]["mixer"]
+    H, G, D, E = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+    RH, RG, RD, RE = d["heads"], d["kv_heads"], d["dim"], d["vdim"]
+    chan = 2 * RG * RD + RH * RE
+    ff = c["layers"][0]["mlp"]["ff"]
+    T, R, Cx = PROMPT, BATCH, PROMPT
+
+    def t_us(by, fl):
+        return max(by / (pk["hbm_gbs"] * 1e9), fl / (pk["bf16_tflops"] * 1e12)) * 1e6
+
+    def both(rows, keys_total, keys_read, requests):
+        proj = (H * D + G * (D + E)) * 2
+        decay = (RH * RD + RH) / 2                # numbers a token, the mean of the two kinds
+        return {
+            "norm_add": t_us(rows * width * (2 + 4 + 4 + 2), 0),
+            "embedding_positions": t_us(rows * width * (2 + 4 + 2), 0),
+            "head_norm_write": t_us(rows * (proj + 4 * H * D + 2 * G * (D + E) + 4 * E), 0),
+            "masked_attention": t_us(4 * rows * H * D + 2 * keys_read * G * (D + E) + 2 * rows * H * E,
+                                     2 * H * (D + E) * keys_total),
+            "gated_activation": t_us(rows * ff * 6, 0),
+            # the projection's columns and the decays' pre-activations in, everything float32 out
+            "delta_inputs": t_us(rows * (2 * chan + 4 * chan + 8 * decay), 0),
+            "delta_scan": t_us(rows * (4 * chan + 4 * decay + 4 * RH * RE) + 8 * requests * RH * RD * RE,
+                               6 * rows * RH * RD * RE),
+            "gated_rms": t_us(rows * RH * RE * (4 + 3 + 2), 0),     # a bfloat16 or a float32 gate
+        }
+    out = {"prefill": both(T, T * (T + 1) // 2, T, 1), "decode": both(R, R * (Cx + 1), R * (Cx + 1), R)}
+    for beside, roofs in (("mobunex", rooflines_mobunex), ("bavetar", rooflines_bavetar)):
+        for phase, kernels in roofs(width, pk).items():
+            out[f"{beside}.{phase}"] = kernels
+    return out
+
+
 def rooflines(width: int, pk: dict):
     """Algorithmic bytes and FLOPs of the compared kernels for the two workloads, per launch."""
     g = gebadra_config(width)
@@ -398,8 +453,9 @@ def run(design: str, steps: int, warmup: int, sizes=(2048, 4096)) -> dict:
     from bench import ClockSampler, peaks
     from paged_batch_engine_b200.config import load_config
     from paged_batch_engine_b200.engine.runner import ModelRunner
-    if design not in ("gebadra", "bavetar", "gusorax", "mobunex"):
-        raise SystemExit(f"unknown design {design!r}; known: gebadra, bavetar, gusorax, mobunex")
+    known = ("gebadra", "bavetar", "gusorax", "mobunex", "tuterax")
+    if design not in known:
+        raise SystemExit(f"unknown design {design!r}; known: {', '.join(known)}")
     os.environ["PBE_EXEC"] = "python"        # per-kernel times need every launch to come through ops
     pk = peaks()
     page = 16
@@ -420,24 +476,29 @@ def run(design: str, steps: int, warmup: int, sizes=(2048, 4096)) -> dict:
     bavetar_ops = ["latent_attention", "head_product", "latent_prepare", "add2_rmsnorm2", "linear_attention",
                    "short_conv", "step_sizes", "gated_rms", "relu_squared", "route", "expert_rows", "expert_places",
                    "expert_gather", "expert_scatter", "grouped_heads", "grouped_runs", "run_tiles"]
-    beside, beside_config = "qwen2", lambda width: qwen_config(width, design)
+    besides = [("qwen2", lambda width: qwen_config(width, design), theirs)]
+    mobunex_ops = ["unit_norm", "embedding_unit_norm", "recurrence_gates", "gated_scan", "short_conv", "masked_attention",
+                   "head_norm_write", "latent_attention", "latent_prepare", "grouped_heads", "silu_mul", "route",
+                   "expert_rows", "expert_places", "expert_gather", "expert_scatter", "grouped_runs", "run_tiles"]
     if design == "mobunex":
-        own = ["unit_norm", "embedding_unit_norm", "recurrence_gates", "gated_scan", "short_conv", "masked_attention",
-               "head_norm_write", "latent_attention", "latent_prepare", "grouped_heads", "silu_mul", "route",
-               "expert_rows", "expert_places", "expert_gather", "expert_scatter", "grouped_runs", "run_tiles"]
-        theirs = bavetar_ops
-        beside, beside_config = "bavetar", bavetar_config
-    design_config = {"bavetar": bavetar_config, "gusorax": gusorax_config, "mobunex": mobunex_config}.get(
-        design, gebadra_config)
-    roofs = {"bavetar": rooflines_bavetar, "gusorax": rooflines_gusorax, "mobunex": rooflines_mobunex}.get(
-        design, rooflines)
+        own = mobunex_ops
+        besides = [("bavetar", bavetar_config, bavetar_ops)]
+    if design == "tuterax":
+        own = ["norm_add", "embedding_positions", "head_norm_write", "masked_attention", "gated_activation",
+               "delta_inputs", "delta_scan", "gated_rms"]
+        besides = [("mobunex", mobunex_config, mobunex_ops), ("bavetar", bavetar_config, bavetar_ops)]
+    design_config = {"bavetar": bavetar_config, "gusorax": gusorax_config, "mobunex": mobunex_config,
+                     "tuterax": tuterax_config}.get(design, gebadra_config)
+    roofs = {"bavetar": rooflines_bavetar, "gusorax": rooflines_gusorax, "mobunex": rooflines_mobunex,
+             "tuterax": rooflines_tuterax}.get(design, rooflines)
     sampler = ClockSampler(0)
     sampler.active = True
     out = {}
     for width in sizes:
         roof = roofs(width, pk)
         row = {}
-        for name, cfg, names in ((design, design_config(width), own), (beside, beside_config(width), theirs)):
+        for name, make, names in [(design, design_config, own)] + besides:
+            cfg = make(width)
             _, typed = load_config(cfg)
             runner = ModelRunner.from_random(typed, seed=0, dtype="bfloat16", page_tokens=page, max_cache_tokens=pool,
                                              max_requests=BATCH + 1)
@@ -445,12 +506,13 @@ def run(design: str, steps: int, warmup: int, sizes=(2048, 4096)) -> dict:
             ms_d, ops_d, captured = _decode(runner, BATCH, PROMPT, steps, warmup, names)
             kernels = {}
             for phase, per_op in (("prefill", ops_p), ("decode", ops_d)):
+                floor = roof.get(f"{name}.{phase}", roof[phase])
                 for op, (ms, calls) in sorted((per_op or {}).items()):
                     us = ms * 1e3 / calls
                     entry = {"us": round(us, 1), "calls": calls}
-                    if op in roof[phase]:
-                        entry["roofline_us"] = round(roof[phase][op], 2)
-                        entry["frac"] = round(roof[phase][op] / us, 4)
+                    if op in floor:
+                        entry["roofline_us"] = round(floor[op], 2)
+                        entry["frac"] = round(floor[op] / us, 4)
                     kernels[f"{phase}.{op}"] = entry
             row[name] = {"prefill_tok_s": round(PROMPT * 1e3 / ms_p, 1), "prefill_ms": round(ms_p, 3),
                          "decode_tok_s": round(BATCH * 1e3 / ms_d, 1), "decode_ms_per_step": round(ms_d, 4),
@@ -461,8 +523,8 @@ def run(design: str, steps: int, warmup: int, sizes=(2048, 4096)) -> dict:
         out[str(width)] = row
     sampler.active = False
     return {"design": design,
-            "beside": f"{beside} at equal width, heads, feed-forward, vocabulary and layers"
-            + (", key/value heads" if beside == "qwen2" else ""),
+            "beside": f"{' and '.join(b[0] for b in besides)} at equal width, heads, feed-forward, vocabulary and layers"
+            + (", key/value heads" if besides[0][0] == "qwen2" else ""),
             "layers": LAYERS, "prompt_tokens": PROMPT, "decode_batch": BATCH, "decode_context": PROMPT,
             "steps": steps, "warmup": warmup, "dtype": "bf16", "data": "synthetic (random weights)",
             "peaks": {"source": pk["source"], "hbm_gbs": pk["hbm_gbs"], "bf16_tflops": pk["bf16_tflops"]},

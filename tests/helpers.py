@@ -456,3 +456,94 @@ def make_mobunex_folder(path, cfg: dict, seed: int, dtype=torch.bfloat16, gain: 
         w[k] = t.to(w[k].dtype)
     save_file(w, f)
     return str(path)
+
+
+# ---------------------------------------------------------------- Tuterax
+def _tatt(heads, kv, dim, vdim, rot_dims, base, scale, softcap):
+    return dict(heads=heads, kv_heads=kv, dim=dim, vdim=vdim, rot=dict(dims=rot_dims, base=base), scale=scale,
+                softcap=softcap)
+
+
+def _tdelta(heads, kv, dim, vdim, conv):
+    return dict(heads=heads, kv_heads=kv, dim=dim, vdim=vdim, conv=conv)
+
+
+# three query heads a key head, values wider than keys, the whole head turns; a decay per channel with two
+# heads a key head and three taps; a decay per head with as many key heads, keys wider than values
+TUT_A = dict(
+    architecture="Tuterax", width=72, vocab=300, norm=dict(eps=1e-5), embedding=dict(scale=1.5),
+    layers=[
+        dict(type="attention", mixer=_tatt(6, 2, 24, 40, 24, 1000.0, 0.2, 8.0), mlp=dict(kind="dense", ff=88)),
+        dict(type="channel_delta", mixer=_tdelta(4, 2, 16, 24, 3), mlp=None),
+        dict(type="delta", mixer=_tdelta(3, 3, 40, 16, 4), mlp=dict(kind="dense", ff=104)),
+        dict(type="attention", mixer=_tatt(2, 2, 12, 6, 2, 50.0, 0.4, 3.0), mlp=None),
+    ])
+# recurrent layers first, one with a single tap (no convolution state); one key head for four heads; heads
+# of 32 and 16 (the tensor-core path in bfloat16), a small cap
+TUT_B = dict(
+    architecture="Tuterax", width=96, vocab=211, norm=dict(eps=1e-6), embedding=dict(scale=0.75),
+    layers=[
+        dict(type="delta", mixer=_tdelta(4, 1, 24, 32, 1), mlp=None),
+        dict(type="attention", mixer=_tatt(5, 5, 32, 16, 4, 300.0, 0.15, 5.0), mlp=dict(kind="dense", ff=64)),
+        dict(type="channel_delta", mixer=_tdelta(3, 3, 8, 8, 2), mlp=dict(kind="dense", ff=72)),
+    ])
+# wide heads (96 keys, 128 values) on one key head; states of more than 128 key channels; head widths that
+# no vector access divides; no cap in one layer; two recurrent layers in a row
+TUT_C = dict(
+    architecture="Tuterax", width=128, vocab=257, norm=dict(eps=1e-6), embedding=dict(scale=4.0),
+    layers=[
+        dict(type="attention", mixer=_tatt(4, 1, 96, 128, 32, 100000.0, 0.06, 20.0), mlp=dict(kind="dense", ff=136)),
+        dict(type="channel_delta", mixer=_tdelta(2, 1, 160, 48, 4), mlp=dict(kind="dense", ff=48)),
+        dict(type="delta", mixer=_tdelta(2, 2, 33, 21, 5), mlp=None),
+        dict(type="attention", mixer=_tatt(3, 3, 16, 32, 8, 20.0, 0.5, None), mlp=None),
+        dict(type="channel_delta", mixer=_tdelta(5, 5, 7, 10, 2), mlp=None),
+    ])
+TUTERAX = {"A": (TUT_A, 81, 8), "B": (TUT_B, 82, 16), "C": (TUT_C, 83, 4)}     # config, seed, page tokens
+
+
+def make_tuterax_folder(path, cfg: dict, seed: int, dtype=torch.bfloat16, gain: float = 1.0, ranks=(12, 20)) -> str:
+    """A model folder with seeded random weights through the engine's random-weights mode, then
+    reshaped so that no mechanism is a near-identity: norm gains far from one, sharp softmaxes with
+    scores near the cap and sinks that matter, decays from almost nothing to almost one, gates and
+    correction strengths spread over their range, low ranks that are no multiple of eight.  ``gain``
+    scales the matrices' factors (wide models need less)."""
+    from paged_batch_engine_b200.config import load_config
+    from paged_batch_engine_b200.engine.runner import build_model
+    from paged_batch_engine_b200.weights import write_random_model
+    from safetensors.torch import load_file, save_file
+    _, typed = load_config(cfg)
+    model = build_model(typed, torch.float32, "cpu")
+    write_random_model(str(path), typed, model.param_specs(), seed, dtype)
+    f = os.path.join(str(path), "model.safetensors")
+    w = load_file(f)
+    g = torch.Generator().manual_seed(seed)
+    for k in list(w):
+        t = w[k].float()
+        leaf = k.split(".mix.")[-1] if ".mix." in k else k.split(".")[-1]
+        if k == "embed":
+            t = t * 25.0
+        elif leaf in ("norm1", "norm2") or k == "final.norm":
+            t = torch.randn(t.shape, generator=g) * 0.3
+        elif leaf == "sink":
+            t = torch.randn(t.shape, generator=g) * 1.5 + 1.0
+        elif leaf in ("q.norm", "k.norm"):
+            t = 0.5 + 2.0 * torch.rand(t.shape, generator=g)
+        elif leaf == "norm":
+            t = 0.5 + torch.rand(t.shape, generator=g)
+        elif leaf.endswith(".conv"):
+            t = torch.randn(t.shape, generator=g) * 0.6
+        elif leaf == "A_log":
+            t = torch.randn(t.shape, generator=g) * 1.0 - 1.5
+        elif leaf == "dt_bias":
+            t = torch.randn(t.shape, generator=g) * 1.5 - 1.0
+        elif leaf in ("a1", "g1"):
+            t = t[:ranks[leaf == "g1"]] * 6.0 * gain
+        elif leaf in ("a2", "g2"):
+            t = t[:, :ranks[leaf == "g2"]] * 25.0 * gain
+        elif leaf in ("a", "b"):
+            t = t * 8.0 * gain
+        elif t.dim() == 2:
+            t = t * 6.0 * gain
+        w[k] = t.to(w[k].dtype).contiguous()
+    save_file(w, f)
+    return str(path)
