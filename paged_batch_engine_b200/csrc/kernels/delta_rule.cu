@@ -18,9 +18,20 @@
 //   S^T q = (g S)^T q + (k . q) u - so one round of shuffles serves both, and a token's dependent
 //   chain is: the lanes' multiply-adds, log2(PARTS) shuffles, u, the update.  Tokens are staged TB at a
 //   time in two shared-memory buffers by cp.async.  The state is laid out [head][column][key channel],
-//   so that the lanes of a column read and write consecutive 16-byte pieces.
-//   A prompt portion and a decoded token take the same path, token by token: how a prompt is cut
-//   changes nothing at all.
+//   so that the lanes of a column read and write consecutive 16-byte pieces.  Steps of single tokens
+//   take this kernel.
+// delta_chunks / delta_scan_chunks: the same recurrence for prompt portions, sixteen tokens of a request at
+//   a time.  With S the state at a chunk's start, kg_j and qg_j token j's key and query times all decays up
+//   to j, kd_j its key times the decays after j, and
+//       L_ji = beta_j k_j . (decays after i up to j) k_i  (i < j),    M_ij = k_i . (decays after i up to j) q_j  (i <= j),
+//   the corrections solve (I + L) u = beta (v - S^T kg), a triangular system of sixteen unknowns whose
+//   matrix belongs to the head, not to the column: delta_chunks inverts it and forms
+//       W = (I + L)^-1 beta kg   and   U = (I + L)^-1 beta v,
+//   so that the scan over chunks is u = U - S^T W, o_j = S^T qg_j + sum_{i<=j} M_ij u_i and
+//   S <- (all decays) S + sum_j kd_j u_j^T: products of small matrices, one round of shuffles for sixteen
+//   tokens.  All decay products are products of numbers in (0, 1], no ratio is formed, so nothing can
+//   overflow; the inverse's entries are bounded by one because every step of the rule is a contraction
+//   for keys of at most unit length.  Everything is float32.
 #include "common.cuh"
 #include "pdl.cuh"
 
@@ -410,6 +421,408 @@ __global__ void __launch_bounds__(32 * WARPS) delta_scan_kernel(ScanParams p) {
   }
 }
 
+// ------------------------------------------------------------------ chunks of sixteen tokens
+constexpr int CH = 16;
+
+// A record holds a chunk of one head: W, QG and KD [CH][DP] each, the chunk's decay product [DP], MQ [CH][CH].
+__host__ __device__ constexpr int record_floats(int dp) { return 3 * CH * dp + dp + CH * CH; }
+// The records of a request that starts at row q of the step: they begin at q / CH + r, which leaves every
+// request room for all its chunks (the last of them may be short) without overlap.
+__device__ __forceinline__ int first_record(int q_start, int r) { return q_start / CH + r; }
+
+struct ChunkParams {
+  const float* qk;           // [T, G, 2, D]
+  const float* decay;        // [T, H] or [T, H * D]
+  const float* beta;         // [T, H]
+  float* v;                  // [T, H * E]: v in, U out
+  float* records;            // [first_record(T, R)][H][record_floats(DP)]
+  const int32_t* q_start;
+  const int32_t* q_len;
+  int R, G, H, D, E;
+};
+
+// grid (records, H), a block of 128 threads a chunk and head
+template <int DP, bool CHAN>
+__global__ void __launch_bounds__(128, 4) delta_chunks_kernel(ChunkParams p) {
+  extern __shared__ __align__(16) float smem[];
+  float* K = smem;                        // [CH][DP]
+  float* Q = K + CH * DP;                 // [CH][DP]
+  float* W = Q + CH * DP;                 // [CH][DP] decays
+  __shared__ float Lk[CH][CH + 1];        // [j][i]: beta_j k_i . (decays after i up to j) k_j, i < j
+  __shared__ __align__(16) float Tb[CH][CH];   // (I + Lk)^-1, columns times beta
+  __shared__ float beta[CH];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int rec = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
+  const int D = p.D, E = p.E, H = p.H, G = p.G;
+  // whose chunk this is
+  int r = -1, c = 0;
+  for (int i = 0; i < p.R; ++i) {
+    const int first = first_record(p.q_start[i], i);
+    if (rec >= first && rec < first + (p.q_len[i] + CH - 1) / CH) {
+      r = i;
+      c = rec - first;
+    }
+  }
+  if (r < 0) return;
+  const int count = min(CH, p.q_len[r] - c * CH);
+  const size_t row0 = (size_t)p.q_start[r] + c * CH;
+  const int g = h / (H / G);
+  for (int i = tid; i < CH * DP; i += 128) {
+    const int j = i / DP, d = i % DP;
+    const bool ok = j < count && d < D;
+    const float* src = p.qk + ((row0 + (ok ? j : 0)) * G + g) * 2 * D + (ok ? d : 0);
+    Q[i] = ok ? src[0] : 0.f;
+    K[i] = ok ? src[D] : 0.f;
+    float w = 1.f;
+    if (j < count) {
+      if (CHAN) w = d < D ? p.decay[((row0 + j) * H + h) * D + d] : 1.f;
+      else w = p.decay[(row0 + j) * H + h];
+    }
+    W[i] = w;
+  }
+  if (tid < CH) beta[tid] = tid < count ? p.beta[(row0 + tid) * H + h] : 0.f;
+  __syncthreads();
+  float* out = p.records + ((size_t)rec * H + h) * record_floats(DP);
+  float* mq = out + 3 * CH * DP + DP;
+  {
+    // eight lanes share a token i, DP / 8 channels each; x runs over k_i times the decays after i
+    constexpr int MPT = DP / 8;
+    const int i = tid >> 3, slice = tid & 7;
+    float x[MPT];
+#pragma unroll
+    for (int m = 0; m < MPT; ++m) x[m] = K[i * DP + slice + 8 * m];
+    for (int j = 0; j < CH; ++j) {
+      float ck = 0.f, cq = 0.f;
+      if (j >= i) {
+#pragma unroll
+        for (int m = 0; m < MPT; ++m) {
+          const int d = j * DP + slice + 8 * m;
+          if (j > i) x[m] *= W[d];
+          ck = fmaf(x[m], K[d], ck);
+          cq = fmaf(x[m], Q[d], cq);
+        }
+      }
+#pragma unroll
+      for (int m = 1; m < 8; m <<= 1) {
+        ck += __shfl_xor_sync(0xffffffffu, ck, m);
+        cq += __shfl_xor_sync(0xffffffffu, cq, m);
+      }
+      if (slice == 0) {
+        Lk[j][i] = j > i ? beta[j] * ck : 0.f;
+        mq[i * CH + j] = j >= i ? cq : 0.f;
+      }
+    }
+    float* kd = out + 2 * CH * DP + i * DP;
+#pragma unroll
+    for (int m = 0; m < MPT; ++m) kd[slice + 8 * m] = x[m];
+  }
+  __syncthreads();
+  if (tid < CH) {                          // a thread a column of the inverse, by substitution
+    float t[CH];
+#pragma unroll
+    for (int j = 0; j < CH; ++j) {
+      float s = j == tid ? 1.f : 0.f;
+#pragma unroll
+      for (int i = 0; i < j; ++i) s = fmaf(-Lk[j][i], t[i], s);      // t[i] is 0 above the diagonal
+      t[j] = s;
+      Tb[j][tid] = s * beta[tid];
+    }
+  }
+  __syncthreads();
+  // rows j of Tb times a column of sixteen numbers
+  auto times_tb = [&](const float (&y)[CH], auto&& put) {
+#pragma unroll
+    for (int j = 0; j < CH; ++j) {
+      float s = 0.f;
+#pragma unroll
+      for (int i = 0; i <= j; i += 4) {
+        const float4 t4 = *reinterpret_cast<const float4*>(&Tb[j][i]);
+        s = fmaf(t4.x, y[i], s);
+        if (i + 1 <= j) s = fmaf(t4.y, y[i + 1], s);
+        if (i + 2 <= j) s = fmaf(t4.z, y[i + 2], s);
+        if (i + 3 <= j) s = fmaf(t4.w, y[i + 3], s);
+      }
+      put(j, s);
+    }
+  };
+  for (int d = tid; d < DP; d += 128) {
+    float kg[CH];
+    float up = 1.f;
+#pragma unroll
+    for (int j = 0; j < CH; ++j) {
+      up *= W[j * DP + d];
+      kg[j] = K[j * DP + d] * up;
+      out[CH * DP + j * DP + d] = Q[j * DP + d] * up;
+    }
+    out[3 * CH * DP + d] = up;
+    times_tb(kg, [&](int j, float s) { out[j * DP + d] = s; });
+  }
+  for (int e = tid; e < E; e += 128) {
+    float y[CH];
+#pragma unroll
+    for (int j = 0; j < CH; ++j) y[j] = j < count ? p.v[((row0 + j) * H + h) * E + e] : 0.f;
+    times_tb(y, [&](int j, float s) {
+      if (j < count) p.v[((row0 + j) * H + h) * E + e] = s;
+    });
+  }
+}
+
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+  f32x2 d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+  f32x2 d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+__device__ __forceinline__ f32x2 pack2(float x, float y) {
+  f32x2 d;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(x), "f"(y));
+  return d;
+}
+__device__ __forceinline__ void unpack2(f32x2 a, float& x, float& y) {
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(a));
+}
+
+struct ChunkScanParams {
+  const float* records;
+  const float* u;            // [T, H * E]
+  float* out;                // [T, H * E]
+  float* state;              // [slots, H, E, D]
+  const int32_t* q_start;
+  const int32_t* q_len;
+  const int32_t* slots;
+  int H, D, E, write_state;
+};
+
+// x: a value per token (16) of each of the sixteen lanes of a half warp; lane p ends with the sum over the
+// lanes of its token p
+__device__ __forceinline__ float scatter_sum(float (&x)[CH], int part) {
+#pragma unroll
+  for (int half = CH / 2; half > 0; half >>= 1) {
+    const bool upper = (part & half) != 0;
+#pragma unroll
+    for (int j = 0; j < half; ++j) {
+      const float mine = upper ? x[j + half] : x[j];
+      const float give = upper ? x[j] : x[j + half];
+      x[j] = mine + __shfl_xor_sync(0xffffffffu, give, half);
+    }
+  }
+  return x[0];
+}
+
+// A half warp shares CPT columns: lane p holds RPT key channels of each (DP = 16 RPT), and stands for the
+// chunk's token p where the chunk's own numbers are concerned.
+template <int RPT, int CPT, int WARPS>
+__global__ void __launch_bounds__(32 * WARPS) delta_scan_chunks_kernel(ChunkScanParams p) {
+  constexpr int NT = 32 * WARPS;
+  constexpr int DP = 16 * RPT;
+  constexpr int QUADS = RPT / 4;
+  constexpr int COLS = 2 * WARPS * CPT;
+  constexpr int REC = record_floats(DP);
+  extern __shared__ __align__(16) float smem[];          // two records
+  pdl_launch_dependents();
+  pdl_wait();
+  const int r = blockIdx.x, h = blockIdx.y;
+  const int tid = threadIdx.x;
+  const int n = p.q_len[r];
+  if (n <= 0) return;
+  const int t0 = p.q_start[r];
+  const int D = p.D, E = p.E, H = p.H;
+  const int part = tid & 15;
+  const int e0 = blockIdx.z * COLS + (tid >> 4) * CPT;   // this half warp's first column
+  const int nc = (n + CH - 1) / CH;
+  const float* rec0 = p.records + ((size_t)first_record(t0, r) * H + h) * REC;
+  auto fetch = [&](int c) {
+    const float* src = rec0 + (size_t)c * H * REC;
+    float* dst = smem + (c & 1) * REC;
+    for (int i = tid; i < REC / 4; i += NT) cp_async16(dst + 4 * i, src + 4 * i);
+  };
+  fetch(0);
+  cp_async_commit();
+  float* st_head = p.state + ((size_t)p.slots[r] * H + h) * E * D;
+  const bool quads = (D & 3) == 0;
+  f32x2 S[CPT][RPT / 2];
+#pragma unroll
+  for (int c = 0; c < CPT; ++c) {
+#pragma unroll
+    for (int j = 0; j < QUADS; ++j) {
+      const int d = (j * 16 + part) * 4;
+      float x[4] = {0.f, 0.f, 0.f, 0.f};
+      if (e0 + c < E) {
+        const float* st = st_head + (size_t)(e0 + c) * D;
+        if (quads && d < D) {
+          const float4 s4 = *reinterpret_cast<const float4*>(st + d);
+          x[0] = s4.x; x[1] = s4.y; x[2] = s4.z; x[3] = s4.w;
+        } else if (!quads) {
+#pragma unroll
+          for (int k = 0; k < 4; ++k)
+            if (d + k < D) x[k] = st[d + k];
+        }
+      }
+      S[c][2 * j] = pack2(x[0], x[1]);
+      S[c][2 * j + 1] = pack2(x[2], x[3]);
+    }
+  }
+  // this lane's token of a chunk: its U in this half warp's columns, requested a chunk ahead
+  float u_next[CPT];
+  auto request_u = [&](int c) {
+    const int t = c * CH + part;
+#pragma unroll
+    for (int k = 0; k < CPT; ++k)
+      u_next[k] = (t < n && e0 + k < E) ? p.u[((size_t)(t0 + t) * H + h) * E + e0 + k] : 0.f;
+  };
+  request_u(0);
+
+#pragma unroll 1
+  for (int c = 0; c < nc; ++c) {
+    cp_async_wait_all();
+    __syncthreads();       // chunk c has landed, chunk c - 1 is computed by all (its buffer is free)
+    if (c + 1 < nc) fetch(c + 1);
+    cp_async_commit();
+    float x[CPT];          // token `part`: U, then u
+#pragma unroll
+    for (int k = 0; k < CPT; ++k) x[k] = u_next[k];
+    if (c + 1 < nc) request_u(c + 1);
+    const float* rec = smem + (c & 1) * REC;
+    // the chunk's products with the state at its start: which = 0: W, 1: QG
+    float dot[2][CPT];
+#pragma unroll
+    for (int which = 0; which < 2; ++which) {
+      f32x2 acc[CPT][CH];
+#pragma unroll
+      for (int k = 0; k < CPT; ++k)
+#pragma unroll
+        for (int j = 0; j < CH; ++j) acc[k][j] = 0ull;
+      const float* base = rec + which * CH * DP + part * 4;
+#pragma unroll
+      for (int j = 0; j < QUADS; ++j) {
+#pragma unroll
+        for (int tt = 0; tt < CH; ++tt) {
+          const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(base + tt * DP + j * 64);
+#pragma unroll
+          for (int k = 0; k < CPT; ++k) {
+            acc[k][tt] = fma2(S[k][2 * j], w.x, acc[k][tt]);
+            acc[k][tt] = fma2(S[k][2 * j + 1], w.y, acc[k][tt]);
+          }
+        }
+      }
+#pragma unroll
+      for (int k = 0; k < CPT; ++k) {
+        float v[CH];
+#pragma unroll
+        for (int tt = 0; tt < CH; ++tt) {
+          float a, b;
+          unpack2(acc[k][tt], a, b);
+          v[tt] = a + b;
+        }
+        dot[which][k] = scatter_sum(v, part);
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < CPT; ++k) x[k] -= dot[0][k];
+    // every lane gets every token's u; the read-outs add what the chunk's own writes give
+    const float* mq = rec + 3 * CH * DP + DP + part;
+    f32x2 u[CPT][CH];
+#pragma unroll
+    for (int i = 0; i < CH; ++i) {
+      const float m = mq[i * CH];
+#pragma unroll
+      for (int k = 0; k < CPT; ++k) {
+        const float ui = __shfl_sync(0xffffffffu, x[k], i, 16);
+        dot[1][k] = fmaf(m, ui, dot[1][k]);
+        u[k][i] = pack2(ui, ui);
+      }
+    }
+    const int t = c * CH + part;
+    if (t < n) {
+      float* o = p.out + ((size_t)(t0 + t) * H + h) * E + e0;
+#pragma unroll
+      for (int k = 0; k < CPT; ++k)
+        if (e0 + k < E) o[k] = dot[1][k];
+    }
+    // S <- decays * S + sum over the tokens of kd u^T
+    const float* kd = rec + 2 * CH * DP + part * 4;
+#pragma unroll
+    for (int j = 0; j < QUADS; ++j) {
+      const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(rec + 3 * CH * DP + part * 4 + j * 64);
+#pragma unroll
+      for (int k = 0; k < CPT; ++k) {
+        S[k][2 * j] = mul2(S[k][2 * j], w.x);
+        S[k][2 * j + 1] = mul2(S[k][2 * j + 1], w.y);
+      }
+#pragma unroll
+      for (int tt = 0; tt < CH; ++tt) {
+        const ulonglong2 y = *reinterpret_cast<const ulonglong2*>(kd + tt * DP + j * 64);
+#pragma unroll
+        for (int k = 0; k < CPT; ++k) {
+          S[k][2 * j] = fma2(y.x, u[k][tt], S[k][2 * j]);
+          S[k][2 * j + 1] = fma2(y.y, u[k][tt], S[k][2 * j + 1]);
+        }
+      }
+    }
+  }
+  if (!p.write_state) return;
+#pragma unroll
+  for (int c = 0; c < CPT; ++c) {
+    if (e0 + c >= E) continue;
+    float* st = st_head + (size_t)(e0 + c) * D;
+#pragma unroll
+    for (int j = 0; j < QUADS; ++j) {
+      const int d = (j * 16 + part) * 4;
+      float x[4];
+      unpack2(S[c][2 * j], x[0], x[1]);
+      unpack2(S[c][2 * j + 1], x[2], x[3]);
+      if (quads && d < D) {
+        *reinterpret_cast<float4*>(st + d) = make_float4(x[0], x[1], x[2], x[3]);
+      } else if (!quads) {
+#pragma unroll
+        for (int k = 0; k < 4; ++k)
+          if (d + k < D) st[d + k] = x[k];
+      }
+    }
+  }
+}
+
+// Launched without the programmatic dependency: its few long-running blocks would else be placed while the
+// kernel before still fills most multiprocessors, several on the same one.
+template <typename... KArgs, typename... Args>
+void launch_spread(void (*kernel)(KArgs...), dim3 grid, int threads, size_t smem, cudaStream_t stream, Args... args) {
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = grid;
+  cfg.blockDim = dim3(threads);
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = stream;
+  cudaLaunchKernelEx(&cfg, kernel, KArgs(args)...);
+}
+
+template <int RPT, int CPT, int WARPS>
+int launch_chunks(const ChunkParams& g, const ChunkScanParams& p, int records, bool chan, cudaStream_t stream) {
+  constexpr int DP = 16 * RPT, COLS = 2 * WARPS * CPT;
+  constexpr size_t smem_g = sizeof(float) * 3 * CH * DP, smem_p = sizeof(float) * 2 * record_floats(DP);
+  static bool opted = false;
+  if (!opted) {
+    cudaFuncSetAttribute(delta_chunks_kernel<DP, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_g);
+    cudaFuncSetAttribute(delta_chunks_kernel<DP, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_g);
+    const cudaError_t e = cudaFuncSetAttribute(delta_scan_chunks_kernel<RPT, CPT, WARPS>,
+                                               cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_p);
+    if (e != cudaSuccess) return (int)e;
+    opted = true;
+  }
+  const dim3 grid(records, g.H);
+  if (chan) launch_k(delta_chunks_kernel<DP, true>, grid, 128, smem_g, stream, g);
+  else launch_k(delta_chunks_kernel<DP, false>, grid, 128, smem_g, stream, g);
+  const int err = launch_status();
+  if (err != 0) return err;
+  launch_spread(delta_scan_chunks_kernel<RPT, CPT, WARPS>, dim3(g.R, g.H, (g.E + COLS - 1) / COLS), 32 * WARPS, smem_p,
+                stream, p);
+  return launch_status();
+}
+
 template <int RPT, int PARTS, int WARPS, int TB>
 void launch_scan(const ScanParams& p, int R, bool chan, cudaStream_t stream) {
   constexpr int COLS = 32 * WARPS / PARTS;
@@ -472,4 +885,28 @@ PBE_EXPORT int pbe_delta_scan(const float* qk, const float* kq, const float* v, 
   else if (D <= MAX_HEAD) launch_scan<16, 32, 4, 2>(p, R, chan, stream);
   else return (int)cudaErrorInvalidValue;
   return launch_status();
+}
+
+// Floats of a chunk's record (a head), for key heads of D channels (0: too wide for the chunked form).
+PBE_EXPORT int pbe_delta_record_floats(int D) {
+  return D <= 64 ? record_floats(64) : D <= 128 ? record_floats(128) : D <= 256 ? record_floats(256) : 0;
+}
+PBE_EXPORT int pbe_delta_chunk_tokens() { return CH; }
+
+// The same for steps with prompt portions, sixteen tokens of a request at a time: two launches.  v is
+// overwritten.  records: [T / 16 + R][H][pbe_delta_record_floats(D)] floats of scratch memory.
+PBE_EXPORT int pbe_delta_scan_chunks(const float* qk, float* v, const float* beta, const float* decay, int per_channel,
+                                     float* out, float* state, float* records, const int32_t* q_start,
+                                     const int32_t* q_len, const int32_t* slots, int T, int R, int G, int H, int D,
+                                     int E, int write_state, cudaStream_t stream) {
+  if (R <= 0 || T <= 0) return 0;
+  if (D < 1 || D > 256 || E < 1 || G < 1 || H % G != 0 || records == nullptr) return (int)cudaErrorInvalidValue;
+  if ((((uintptr_t)state | (uintptr_t)records) & 15) != 0) return (int)cudaErrorMisalignedAddress;
+  const ChunkParams g{qk, decay, beta, v, records, q_start, q_len, R, G, H, D, E};
+  const ChunkScanParams p{records, v, out, state, q_start, q_len, slots, H, D, E, write_state};
+  const int n = T / CH + R;
+  const bool chan = per_channel != 0;
+  if (D <= 64) return launch_chunks<4, 2, 4>(g, p, n, chan, stream);
+  if (D <= 128) return launch_chunks<8, 2, 4>(g, p, n, chan, stream);
+  return launch_chunks<16, 2, 4>(g, p, n, chan, stream);
 }

@@ -2063,13 +2063,18 @@ def delta_inputs(proj: torch.Tensor, conv_t: torch.Tensor, conv_state: torch.Ten
     return qk, kq, v, beta, decay
 
 
+DELTA_CHUNK_MAX_DIM = 256     # wider key heads always run token by token
+
+
 def delta_scan(qk: torch.Tensor, kq: torch.Tensor, v: torch.Tensor, beta: torch.Tensor, decay: torch.Tensor,
                state: torch.Tensor, q_start: torch.Tensor, q_len: torch.Tensor, slots: torch.Tensor, num_requests: int,
-               update_state: bool = True, zero_out: bool = False) -> torch.Tensor:
+               update_state: bool = True, zero_out: bool = False,
+               chunked: bool = False) -> torch.Tensor:
     """The gated delta rule request by request over the rows each brings: S <- g S,
     u = beta (v - S^T k), S <- S + k u^T, o = S^T q, with the inputs of ``delta_inputs`` and ``state``
     float32 [slots, H, E, D] (S transposed: a value column's key channels side by side), read at
-    ``slots[r]`` and left updated.  Returns o, float32 [T, H * E]."""
+    ``slots[r]`` and left updated.  ``chunked``: sixteen tokens at a time
+    (prompt portions: two launches, v is overwritten), else one by one.  Returns o, float32 [T, H * E]."""
     _need_cuda(qk, kq, v, beta, decay, state, q_start, q_len, slots)
     _need_contiguous(qk, kq, v, beta, decay, state)
     T, G, _, D = qk.shape
@@ -2086,6 +2091,17 @@ def delta_scan(qk: torch.Tensor, kq: torch.Tensor, v: torch.Tensor, beta: torch.
             raise KernelError("delta_scan: request arrays are int32 [R]")
     per_channel = decay.shape[1] == H * D and D > 1
     out = (torch.zeros if zero_out else torch.empty)((T, H * E), dtype=torch.float32, device=v.device)
+    if chunked and D <= DELTA_CHUNK_MAX_DIM:
+        size = _fn("delta_rule", "pbe_delta_record_floats", [c_int])(D)
+        ct = _fn("delta_rule", "pbe_delta_chunk_tokens", [])()
+        records = torch.empty((T // ct + int(num_requests), H, size), dtype=torch.float32, device=v.device)
+        fn = _fn("delta_rule", "pbe_delta_scan_chunks", [c_void_p] * 4 + [c_int] + [c_void_p] * 6 + [c_int] * 7 + [c_void_p])
+        global _launches
+        _check(fn(_ptr(qk), _ptr(v), _ptr(beta), _ptr(decay), 1 if per_channel else 0, _ptr(out), _ptr(state),
+                  _ptr(records), _ptr(q_start), _ptr(q_len), _ptr(slots), T, int(num_requests), G, H, D, E,
+                  1 if update_state else 0, _stream()), "delta_scan_chunks")
+        _launches += 1
+        return out
     fn = _fn("delta_rule", "pbe_delta_scan", [c_void_p] * 5 + [c_int] + [c_void_p] * 5 + [c_int] * 6 + [c_void_p])
     _check(fn(_ptr(qk), _ptr(kq), _ptr(v), _ptr(beta), _ptr(decay), 1 if per_channel else 0, _ptr(out), _ptr(state),
               _ptr(q_start), _ptr(q_len), _ptr(slots), int(num_requests), G, H, D, E, 1 if update_state else 0,

@@ -153,13 +153,15 @@ class GatedDeltaRule(Mixer):
         else:
             conv_state = torch.empty((1, 0, self.channels), dtype=torch.float32, device=x.device)
         captured = getattr(ctx, "captured", False)
+        single = captured or ctx.num_tokens == ctx.num_requests        # every request brings one token
         qk, kq, v, beta, decay = ops.delta_inputs(
             proj, self.conv_t, conv_state, small, wide[:, :H * D] if self.decay == "channel" else None, self.dt_bias,
             self.a_log, ctx.request_of_row, ctx.q_start, ctx.q_len, ctx.state_slots, ctx.num_requests, G, H, D, E,
             D ** -0.5, self.unit_eps, update_state=cache.writes,
-            single_tokens=captured or ctx.num_tokens == ctx.num_requests)
+            single_tokens=single)
         o = ops.delta_scan(qk, kq, v, beta, decay, cache.sub["delta"].state, ctx.q_start, ctx.q_len, ctx.state_slots,
-                           ctx.num_requests, update_state=cache.writes, zero_out=captured)
+                           ctx.num_requests, update_state=cache.writes, zero_out=captured,
+                           chunked=not single)
         y = ops.gated_rms(o, gate, self.gain, H, self.eps, True, self.gate, self.dtype)
         return ops.linear(y, self.w_o, None, out_dtype=self.dtype, kind=2)
 

@@ -168,15 +168,17 @@ def _scan_case(T, G, H, D, E, channel, g):
     return q, k, v, beta, decay
 
 
+@pytest.mark.parametrize("chunked", [False, True])
 @pytest.mark.parametrize("channel", [False, True])
 @pytest.mark.parametrize("G, H, D, E", [(1, 2, 5, 3), (2, 2, 16, 20), (1, 3, 33, 21), (2, 4, 64, 40), (1, 1, 100, 17),
-                                        (1, 2, 130, 32), (1, 1, 300, 18), (1, 1, 512, 5)])
-def test_delta_scan_carries_its_state(G, H, D, E, channel):
-    """Unequal requests in one launch, cut into launches at arbitrary places, on state rows that
+                                        (1, 2, 130, 32), (1, 1, 300, 18), (1, 1, 512, 5),
+                                        (2, 2, 128, 128), (1, 1, 254, 36)])
+def test_delta_scan_carries_its_state(G, H, D, E, channel, chunked):
+    """Token by token and sixteen tokens at a time.  Unequal requests in one launch, cut into launches at arbitrary places, on state rows that
     hold someone else's numbers until they are zeroed; the other rows are left alone."""
     ops = _ops()
     g = torch.Generator().manual_seed(D + E)
-    lens, slots = [1, 29, 0, 16], [3, 0, 4, 1]
+    lens, slots = [1, 69, 0, 33], [3, 0, 4, 1]
     state = torch.full((6, H, E, D), 3.0, device=DEV)
     data, want = [], []
     for n, s in zip(lens, slots):
@@ -189,14 +191,15 @@ def test_delta_scan_carries_its_state(G, H, D, E, channel):
         data.append((q, k, v, beta, decay))
     outs = [[] for _ in lens]
     done = [0] * 4
-    for counts in ([1, 8, 0, 3], [0, 2, 0, 2], [0, 19, 0, 11]):
+    for counts in ([1, 8, 0, 17], [0, 2, 0, 0], [0, 59, 0, 16]):
         parts = [tuple(x[d:d + c] for x in row) for row, d, c in zip(data, done, counts)]
         q, k, v, beta, decay = (torch.cat([p[j] for p in parts]) for j in range(5))
         T = q.shape[0]
         starts = [sum(counts[:i]) for i in range(4)]
         got = ops.delta_scan(torch.stack([q, k], dim=2).contiguous().to(DEV), (q * k).sum(-1).to(DEV),
                              v.reshape(T, H * E).to(DEV), beta.to(DEV), decay.reshape(T, -1).contiguous().to(DEV), state,
-                             i32(starts), i32(counts), i32(slots), 4).cpu()
+                             i32(starts), i32(counts), i32(slots), 4,
+                             chunked=chunked).cpu()
         for r in range(4):
             outs[r].append(got[starts[r]:starts[r] + counts[r]])
             done[r] += counts[r]
