@@ -455,31 +455,52 @@ __global__ void __launch_bounds__(128, 4) delta_chunks_kernel(ChunkParams p) {
   pdl_wait();
   const int rec = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
   const int D = p.D, E = p.E, H = p.H, G = p.G;
-  // whose chunk this is
-  int r = -1, c = 0;
-  for (int i = 0; i < p.R; ++i) {
+  // whose chunk this is: each thread looks at some of the requests, one of them finds it
+  __shared__ int owner;
+  if (tid == 0) owner = -1;
+  __syncthreads();
+  for (int i = tid; i < p.R; i += 128) {
     const int first = first_record(p.q_start[i], i);
-    if (rec >= first && rec < first + (p.q_len[i] + CH - 1) / CH) {
-      r = i;
-      c = rec - first;
-    }
+    if (rec >= first && rec < first + (p.q_len[i] + CH - 1) / CH) owner = i;
   }
+  __syncthreads();
+  const int r = owner;
   if (r < 0) return;
+  const int c = rec - first_record(p.q_start[r], r);
   const int count = min(CH, p.q_len[r] - c * CH);
   const size_t row0 = (size_t)p.q_start[r] + c * CH;
   const int g = h / (H / G);
-  for (int i = tid; i < CH * DP; i += 128) {
-    const int j = i / DP, d = i % DP;
-    const bool ok = j < count && d < D;
-    const float* src = p.qk + ((row0 + (ok ? j : 0)) * G + g) * 2 * D + (ok ? d : 0);
-    Q[i] = ok ? src[0] : 0.f;
-    K[i] = ok ? src[D] : 0.f;
-    float w = 1.f;
-    if (j < count) {
-      if (CHAN) w = d < D ? p.decay[((row0 + j) * H + h) * D + d] : 1.f;
-      else w = p.decay[(row0 + j) * H + h];
+  if ((D & 3) == 0) {                     // sixteen bytes a load, all of a thread's loads in flight
+#pragma unroll
+    for (int n = 0; n < CH * DP / 512; ++n) {
+      const int i = (tid + n * 128) * 4;
+      const int j = i / DP, d = i % DP;
+      const bool ok = j < count && d < D;
+      float4 q4 = make_float4(0.f, 0.f, 0.f, 0.f), k4 = q4, w4 = make_float4(1.f, 1.f, 1.f, 1.f);
+      if (ok) {
+        const float* src = p.qk + ((row0 + j) * G + g) * 2 * D + d;
+        q4 = *reinterpret_cast<const float4*>(src);
+        k4 = *reinterpret_cast<const float4*>(src + D);
+        if (CHAN) {
+          w4 = *reinterpret_cast<const float4*>(p.decay + ((row0 + j) * H + h) * D + d);
+        } else {
+          const float w = p.decay[(row0 + j) * H + h];
+          w4 = make_float4(w, w, w, w);
+        }
+      }
+      *reinterpret_cast<float4*>(Q + i) = q4;
+      *reinterpret_cast<float4*>(K + i) = k4;
+      *reinterpret_cast<float4*>(W + i) = w4;
     }
-    W[i] = w;
+  } else {
+    for (int i = tid; i < CH * DP; i += 128) {
+      const int j = i / DP, d = i % DP;
+      const bool ok = j < count && d < D;
+      const float* src = p.qk + ((row0 + (ok ? j : 0)) * G + g) * 2 * D + (ok ? d : 0);
+      Q[i] = ok ? src[0] : 0.f;
+      K[i] = ok ? src[D] : 0.f;
+      W[i] = ok ? (CHAN ? p.decay[((row0 + j) * H + h) * D + d] : p.decay[(row0 + j) * H + h]) : 1.f;
+    }
   }
   if (tid < CH) beta[tid] = tid < count ? p.beta[(row0 + tid) * H + h] : 0.f;
   __syncthreads();
@@ -902,6 +923,8 @@ PBE_EXPORT int pbe_delta_scan_chunks(const float* qk, float* v, const float* bet
   if (R <= 0 || T <= 0) return 0;
   if (D < 1 || D > 256 || E < 1 || G < 1 || H % G != 0 || records == nullptr) return (int)cudaErrorInvalidValue;
   if ((((uintptr_t)state | (uintptr_t)records) & 15) != 0) return (int)cudaErrorMisalignedAddress;
+  if ((D & 3) == 0 && (((uintptr_t)qk | (per_channel ? (uintptr_t)decay : 0)) & 15) != 0)
+    return (int)cudaErrorMisalignedAddress;
   const ChunkParams g{qk, decay, beta, v, records, q_start, q_len, R, G, H, D, E};
   const ChunkScanParams p{records, v, out, state, q_start, q_len, slots, H, D, E, write_state};
   const int n = T / CH + R;
