@@ -20,7 +20,7 @@
 //   time in two shared-memory buffers by cp.async.  The state is laid out [head][column][key channel],
 //   so that the lanes of a column read and write consecutive 16-byte pieces.  Steps of single tokens
 //   take this kernel.
-// delta_chunks / delta_scan_chunks: the same recurrence for prompt portions, sixteen tokens of a request at
+// delta_chunks and the scan of chunk_scan.cuh: the same recurrence for prompt portions, sixteen tokens of a request at
 //   a time.  With S the state at a chunk's start, kg_j and qg_j token j's key and query times all decays up
 //   to j, kd_j its key times the decays after j, and
 //       L_ji = beta_j k_j . (decays after i up to j) k_i  (i < j),    M_ij = k_i . (decays after i up to j) q_j  (i <= j),
@@ -32,6 +32,7 @@
 //   tokens.  All decay products are products of numbers in (0, 1], no ratio is formed, so nothing can
 //   overflow; the inverse's entries are bounded by one because every step of the rule is a contraction
 //   for keys of at most unit length.  Everything is float32.
+#include "chunk_scan.cuh"
 #include "common.cuh"
 #include "pdl.cuh"
 
@@ -67,32 +68,6 @@ struct InputParams {
 
 __device__ __forceinline__ float softplus_(float x) { return x > 20.f ? x : log1pf(expf(x)); }
 
-template <int V>
-__device__ __forceinline__ void load_v(const float* p, float (&a)[V]) {
-  if constexpr (V == 4) {
-    const float4 v = *reinterpret_cast<const float4*>(p);
-    a[0] = v.x; a[1] = v.y; a[2] = v.z; a[3] = v.w;
-  } else {
-    a[0] = *p;
-  }
-}
-template <int V>
-__device__ __forceinline__ void load_v(const __nv_bfloat16* p, float (&a)[V]) {
-  if constexpr (V == 4) {
-    const uint2 raw = *reinterpret_cast<const uint2*>(p);
-    const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
-    const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
-    a[0] = lo.x; a[1] = lo.y; a[2] = hi.x; a[3] = hi.y;
-  } else {
-    a[0] = __bfloat162float(*p);
-  }
-}
-template <int V>
-__device__ __forceinline__ void store_v(float* p, const float (&a)[V]) {
-  if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(a[0], a[1], a[2], a[3]);
-  else *p = a[0];
-}
-
 // The convolution of V neighbouring channels from column c of one token, with silu.
 template <typename T, int V>
 __device__ __forceinline__ void conv_silu(const InputParams& p, int t, int i, const float* st_in, float* st_out, int C,
@@ -109,7 +84,7 @@ __device__ __forceinline__ void conv_silu(const InputParams& p, int t, int i, co
     load_v<V>(p.conv_t + (size_t)j * C + c, w);
 #pragma unroll
     for (int k = 0; k < V; ++k) acc[k] = fmaf(w[k], u[k], acc[k]);
-    if (st_out && j > 0) store_v<V>(st_out + (size_t)(j - 1) * C + c, u);     // entry j - 1 was read the turn before
+    if (st_out && j > 0) put_v<V>(st_out + (size_t)(j - 1) * C + c, u);     // entry j - 1 was read the turn before
   }
 #pragma unroll
   for (int k = 0; k < V; ++k) acc[k] = acc[k] / (1.0f + expf(-acc[k]));
@@ -183,8 +158,8 @@ __global__ void __launch_bounds__(IN_WARPS * 32) delta_inputs_kernel(InputParams
         dot = fmaf(q[n][e], k[n][e], dot);
       }
       if (d < D) {
-        store_v<V>(out + d, q[n]);
-        store_v<V>(out + D + d, k[n]);
+        put_v<V>(out + d, q[n]);
+        put_v<V>(out + D + d, k[n]);
       }
     }
     dot = warp_sum(dot);
@@ -199,7 +174,7 @@ __global__ void __launch_bounds__(IN_WARPS * 32) delta_inputs_kernel(InputParams
 #pragma unroll
         for (int k = 0; k < V; ++k) v[k] = 0.f;
         if (live) conv_silu<T, V>(p, t, i, st, st_out, C, 2 * G * D + h * E + e, v);
-        store_v<V>(p.v + (size_t)t * H * E + h * E + e, v);
+        put_v<V>(p.v + (size_t)t * H * E + h * E + e, v);
       }
     }
   }
@@ -239,17 +214,6 @@ struct ScanParams {
   const int32_t* slots;
   int G, H, D, E, write_state;
 };
-
-__device__ __forceinline__ void cp_async16(void* smem, const void* gmem) {
-  const unsigned s = (unsigned)__cvta_generic_to_shared(smem);
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(s), "l"(gmem));
-}
-__device__ __forceinline__ void cp_async4(void* smem, const void* gmem) {
-  const unsigned s = (unsigned)__cvta_generic_to_shared(smem);
-  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"(s), "l"(gmem));
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;\n" ::); }
-__device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_group 0;\n" ::); }
 
 template <int RPT, int PARTS, int WARPS, int TB, bool CHAN>
 __global__ void __launch_bounds__(32 * WARPS) delta_scan_kernel(ScanParams p) {
@@ -422,14 +386,6 @@ __global__ void __launch_bounds__(32 * WARPS) delta_scan_kernel(ScanParams p) {
 }
 
 // ------------------------------------------------------------------ chunks of sixteen tokens
-constexpr int CH = 16;
-
-// A record holds a chunk of one head: W, QG and KD [CH][DP] each, the chunk's decay product [DP], MQ [CH][CH].
-__host__ __device__ constexpr int record_floats(int dp) { return 3 * CH * dp + dp + CH * CH; }
-// The records of a request that starts at row q of the step: they begin at q / CH + r, which leaves every
-// request room for all its chunks (the last of them may be short) without overlap.
-__device__ __forceinline__ int first_record(int q_start, int r) { return q_start / CH + r; }
-
 struct ChunkParams {
   const float* qk;           // [T, G, 2, D]
   const float* decay;        // [T, H] or [T, H * D]
@@ -455,16 +411,7 @@ __global__ void __launch_bounds__(128, 4) delta_chunks_kernel(ChunkParams p) {
   pdl_wait();
   const int rec = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
   const int D = p.D, E = p.E, H = p.H, G = p.G;
-  // whose chunk this is: each thread looks at some of the requests, one of them finds it
-  __shared__ int owner;
-  if (tid == 0) owner = -1;
-  __syncthreads();
-  for (int i = tid; i < p.R; i += 128) {
-    const int first = first_record(p.q_start[i], i);
-    if (rec >= first && rec < first + (p.q_len[i] + CH - 1) / CH) owner = i;
-  }
-  __syncthreads();
-  const int r = owner;
+  const int r = record_owner<128>(rec, p.q_start, p.q_len, p.R);
   if (r < 0) return;
   const int c = rec - first_record(p.q_start[r], r);
   const int count = min(CH, p.q_len[r] - c * CH);
@@ -504,8 +451,8 @@ __global__ void __launch_bounds__(128, 4) delta_chunks_kernel(ChunkParams p) {
   }
   if (tid < CH) beta[tid] = tid < count ? p.beta[(row0 + tid) * H + h] : 0.f;
   __syncthreads();
-  float* out = p.records + ((size_t)rec * H + h) * record_floats(DP);
-  float* mq = out + 3 * CH * DP + DP;
+  float* out = p.records + ((size_t)rec * H + h) * record_floats(DP, true);
+  float* mq = out + rec_mq(DP);
   {
     // eight lanes share a token i, DP / 8 channels each; x runs over k_i times the decays after i
     constexpr int MPT = DP / 8;
@@ -534,7 +481,7 @@ __global__ void __launch_bounds__(128, 4) delta_chunks_kernel(ChunkParams p) {
         mq[i * CH + j] = j >= i ? cq : 0.f;
       }
     }
-    float* kd = out + 2 * CH * DP + i * DP;
+    float* kd = out + rec_kd(DP) + i * DP;
 #pragma unroll
     for (int m = 0; m < MPT; ++m) kd[slice + 8 * m] = x[m];
   }
@@ -574,10 +521,10 @@ __global__ void __launch_bounds__(128, 4) delta_chunks_kernel(ChunkParams p) {
     for (int j = 0; j < CH; ++j) {
       up *= W[j * DP + d];
       kg[j] = K[j * DP + d] * up;
-      out[CH * DP + j * DP + d] = Q[j * DP + d] * up;
+      out[j * DP + d] = Q[j * DP + d] * up;
     }
-    out[3 * CH * DP + d] = up;
-    times_tb(kg, [&](int j, float s) { out[j * DP + d] = s; });
+    out[rec_decay(DP) + d] = up;
+    times_tb(kg, [&](int j, float s) { out[rec_w(DP) + j * DP + d] = s; });
   }
   for (int e = tid; e < E; e += 128) {
     float y[CH];
@@ -589,247 +536,15 @@ __global__ void __launch_bounds__(128, 4) delta_chunks_kernel(ChunkParams p) {
   }
 }
 
-typedef unsigned long long f32x2;
-__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
-  f32x2 d;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-  return d;
-}
-__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
-  f32x2 d;
-  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
-  return d;
-}
-__device__ __forceinline__ f32x2 pack2(float x, float y) {
-  f32x2 d;
-  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(x), "f"(y));
-  return d;
-}
-__device__ __forceinline__ void unpack2(f32x2 a, float& x, float& y) {
-  asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(a));
-}
-
-struct ChunkScanParams {
-  const float* records;
-  const float* u;            // [T, H * E]
-  float* out;                // [T, H * E]
-  float* state;              // [slots, H, E, D]
-  const int32_t* q_start;
-  const int32_t* q_len;
-  const int32_t* slots;
-  int H, D, E, write_state;
-};
-
-// x: a value per token (16) of each of the sixteen lanes of a half warp; lane p ends with the sum over the
-// lanes of its token p
-__device__ __forceinline__ float scatter_sum(float (&x)[CH], int part) {
-#pragma unroll
-  for (int half = CH / 2; half > 0; half >>= 1) {
-    const bool upper = (part & half) != 0;
-#pragma unroll
-    for (int j = 0; j < half; ++j) {
-      const float mine = upper ? x[j + half] : x[j];
-      const float give = upper ? x[j] : x[j + half];
-      x[j] = mine + __shfl_xor_sync(0xffffffffu, give, half);
-    }
-  }
-  return x[0];
-}
-
-// A half warp shares CPT columns: lane p holds RPT key channels of each (DP = 16 RPT), and stands for the
-// chunk's token p where the chunk's own numbers are concerned.
 template <int RPT, int CPT, int WARPS>
-__global__ void __launch_bounds__(32 * WARPS) delta_scan_chunks_kernel(ChunkScanParams p) {
-  constexpr int NT = 32 * WARPS;
-  constexpr int DP = 16 * RPT;
-  constexpr int QUADS = RPT / 4;
-  constexpr int COLS = 2 * WARPS * CPT;
-  constexpr int REC = record_floats(DP);
-  extern __shared__ __align__(16) float smem[];          // two records
-  pdl_launch_dependents();
-  pdl_wait();
-  const int r = blockIdx.x, h = blockIdx.y;
-  const int tid = threadIdx.x;
-  const int n = p.q_len[r];
-  if (n <= 0) return;
-  const int t0 = p.q_start[r];
-  const int D = p.D, E = p.E, H = p.H;
-  const int part = tid & 15;
-  const int e0 = blockIdx.z * COLS + (tid >> 4) * CPT;   // this half warp's first column
-  const int nc = (n + CH - 1) / CH;
-  const float* rec0 = p.records + ((size_t)first_record(t0, r) * H + h) * REC;
-  auto fetch = [&](int c) {
-    const float* src = rec0 + (size_t)c * H * REC;
-    float* dst = smem + (c & 1) * REC;
-    for (int i = tid; i < REC / 4; i += NT) cp_async16(dst + 4 * i, src + 4 * i);
-  };
-  fetch(0);
-  cp_async_commit();
-  float* st_head = p.state + ((size_t)p.slots[r] * H + h) * E * D;
-  const bool quads = (D & 3) == 0;
-  f32x2 S[CPT][RPT / 2];
-#pragma unroll
-  for (int c = 0; c < CPT; ++c) {
-#pragma unroll
-    for (int j = 0; j < QUADS; ++j) {
-      const int d = (j * 16 + part) * 4;
-      float x[4] = {0.f, 0.f, 0.f, 0.f};
-      if (e0 + c < E) {
-        const float* st = st_head + (size_t)(e0 + c) * D;
-        if (quads && d < D) {
-          const float4 s4 = *reinterpret_cast<const float4*>(st + d);
-          x[0] = s4.x; x[1] = s4.y; x[2] = s4.z; x[3] = s4.w;
-        } else if (!quads) {
-#pragma unroll
-          for (int k = 0; k < 4; ++k)
-            if (d + k < D) x[k] = st[d + k];
-        }
-      }
-      S[c][2 * j] = pack2(x[0], x[1]);
-      S[c][2 * j + 1] = pack2(x[2], x[3]);
-    }
-  }
-  // this lane's token of a chunk: its U in this half warp's columns, requested a chunk ahead
-  float u_next[CPT];
-  auto request_u = [&](int c) {
-    const int t = c * CH + part;
-#pragma unroll
-    for (int k = 0; k < CPT; ++k)
-      u_next[k] = (t < n && e0 + k < E) ? p.u[((size_t)(t0 + t) * H + h) * E + e0 + k] : 0.f;
-  };
-  request_u(0);
-
-#pragma unroll 1
-  for (int c = 0; c < nc; ++c) {
-    cp_async_wait_all();
-    __syncthreads();       // chunk c has landed, chunk c - 1 is computed by all (its buffer is free)
-    if (c + 1 < nc) fetch(c + 1);
-    cp_async_commit();
-    float x[CPT];          // token `part`: U, then u
-#pragma unroll
-    for (int k = 0; k < CPT; ++k) x[k] = u_next[k];
-    if (c + 1 < nc) request_u(c + 1);
-    const float* rec = smem + (c & 1) * REC;
-    // the chunk's products with the state at its start: which = 0: W, 1: QG
-    float dot[2][CPT];
-#pragma unroll
-    for (int which = 0; which < 2; ++which) {
-      f32x2 acc[CPT][CH];
-#pragma unroll
-      for (int k = 0; k < CPT; ++k)
-#pragma unroll
-        for (int j = 0; j < CH; ++j) acc[k][j] = 0ull;
-      const float* base = rec + which * CH * DP + part * 4;
-#pragma unroll
-      for (int j = 0; j < QUADS; ++j) {
-#pragma unroll
-        for (int tt = 0; tt < CH; ++tt) {
-          const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(base + tt * DP + j * 64);
-#pragma unroll
-          for (int k = 0; k < CPT; ++k) {
-            acc[k][tt] = fma2(S[k][2 * j], w.x, acc[k][tt]);
-            acc[k][tt] = fma2(S[k][2 * j + 1], w.y, acc[k][tt]);
-          }
-        }
-      }
-#pragma unroll
-      for (int k = 0; k < CPT; ++k) {
-        float v[CH];
-#pragma unroll
-        for (int tt = 0; tt < CH; ++tt) {
-          float a, b;
-          unpack2(acc[k][tt], a, b);
-          v[tt] = a + b;
-        }
-        dot[which][k] = scatter_sum(v, part);
-      }
-    }
-#pragma unroll
-    for (int k = 0; k < CPT; ++k) x[k] -= dot[0][k];
-    // every lane gets every token's u; the read-outs add what the chunk's own writes give
-    const float* mq = rec + 3 * CH * DP + DP + part;
-    f32x2 u[CPT][CH];
-#pragma unroll
-    for (int i = 0; i < CH; ++i) {
-      const float m = mq[i * CH];
-#pragma unroll
-      for (int k = 0; k < CPT; ++k) {
-        const float ui = __shfl_sync(0xffffffffu, x[k], i, 16);
-        dot[1][k] = fmaf(m, ui, dot[1][k]);
-        u[k][i] = pack2(ui, ui);
-      }
-    }
-    const int t = c * CH + part;
-    if (t < n) {
-      float* o = p.out + ((size_t)(t0 + t) * H + h) * E + e0;
-#pragma unroll
-      for (int k = 0; k < CPT; ++k)
-        if (e0 + k < E) o[k] = dot[1][k];
-    }
-    // S <- decays * S + sum over the tokens of kd u^T
-    const float* kd = rec + 2 * CH * DP + part * 4;
-#pragma unroll
-    for (int j = 0; j < QUADS; ++j) {
-      const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(rec + 3 * CH * DP + part * 4 + j * 64);
-#pragma unroll
-      for (int k = 0; k < CPT; ++k) {
-        S[k][2 * j] = mul2(S[k][2 * j], w.x);
-        S[k][2 * j + 1] = mul2(S[k][2 * j + 1], w.y);
-      }
-#pragma unroll
-      for (int tt = 0; tt < CH; ++tt) {
-        const ulonglong2 y = *reinterpret_cast<const ulonglong2*>(kd + tt * DP + j * 64);
-#pragma unroll
-        for (int k = 0; k < CPT; ++k) {
-          S[k][2 * j] = fma2(y.x, u[k][tt], S[k][2 * j]);
-          S[k][2 * j + 1] = fma2(y.y, u[k][tt], S[k][2 * j + 1]);
-        }
-      }
-    }
-  }
-  if (!p.write_state) return;
-#pragma unroll
-  for (int c = 0; c < CPT; ++c) {
-    if (e0 + c >= E) continue;
-    float* st = st_head + (size_t)(e0 + c) * D;
-#pragma unroll
-    for (int j = 0; j < QUADS; ++j) {
-      const int d = (j * 16 + part) * 4;
-      float x[4];
-      unpack2(S[c][2 * j], x[0], x[1]);
-      unpack2(S[c][2 * j + 1], x[2], x[3]);
-      if (quads && d < D) {
-        *reinterpret_cast<float4*>(st + d) = make_float4(x[0], x[1], x[2], x[3]);
-      } else if (!quads) {
-#pragma unroll
-        for (int k = 0; k < 4; ++k)
-          if (d + k < D) st[d + k] = x[k];
-      }
-    }
-  }
-}
-
-// Launched without the programmatic dependency: its few long-running blocks would else be placed while the
-// kernel before still fills most multiprocessors, several on the same one.
-template <typename... KArgs, typename... Args>
-void launch_spread(void (*kernel)(KArgs...), dim3 grid, int threads, size_t smem, cudaStream_t stream, Args... args) {
-  cudaLaunchConfig_t cfg = {};
-  cfg.gridDim = grid;
-  cfg.blockDim = dim3(threads);
-  cfg.dynamicSmemBytes = smem;
-  cfg.stream = stream;
-  cudaLaunchKernelEx(&cfg, kernel, KArgs(args)...);
-}
-
-template <int RPT, int CPT, int WARPS>
-int launch_chunks(const ChunkParams& g, const ChunkScanParams& p, int records, bool chan, cudaStream_t stream) {
+int launch_chunks(const ChunkParams& g, const ChunkScanParams<float>& p, int records, bool chan, cudaStream_t stream) {
   constexpr int DP = 16 * RPT, COLS = 2 * WARPS * CPT;
-  constexpr size_t smem_g = sizeof(float) * 3 * CH * DP, smem_p = sizeof(float) * 2 * record_floats(DP);
+  constexpr size_t smem_g = sizeof(float) * 3 * CH * DP, smem_p = sizeof(float) * 2 * record_floats(DP, true);
   static bool opted = false;
   if (!opted) {
     cudaFuncSetAttribute(delta_chunks_kernel<DP, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_g);
     cudaFuncSetAttribute(delta_chunks_kernel<DP, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_g);
-    const cudaError_t e = cudaFuncSetAttribute(delta_scan_chunks_kernel<RPT, CPT, WARPS>,
+    const cudaError_t e = cudaFuncSetAttribute(scan_chunks_kernel<RPT, CPT, WARPS, true, float>,
                                                cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_p);
     if (e != cudaSuccess) return (int)e;
     opted = true;
@@ -839,7 +554,7 @@ int launch_chunks(const ChunkParams& g, const ChunkScanParams& p, int records, b
   else launch_k(delta_chunks_kernel<DP, false>, grid, 128, smem_g, stream, g);
   const int err = launch_status();
   if (err != 0) return err;
-  launch_spread(delta_scan_chunks_kernel<RPT, CPT, WARPS>, dim3(g.R, g.H, (g.E + COLS - 1) / COLS), 32 * WARPS, smem_p,
+  launch_spread(scan_chunks_kernel<RPT, CPT, WARPS, true, float>, dim3(g.R, g.H, (g.E + COLS - 1) / COLS), 32 * WARPS, smem_p,
                 stream, p);
   return launch_status();
 }
@@ -910,7 +625,7 @@ PBE_EXPORT int pbe_delta_scan(const float* qk, const float* kq, const float* v, 
 
 // Floats of a chunk's record (a head), for key heads of D channels (0: too wide for the chunked form).
 PBE_EXPORT int pbe_delta_record_floats(int D) {
-  return D <= 64 ? record_floats(64) : D <= 128 ? record_floats(128) : D <= 256 ? record_floats(256) : 0;
+  return D <= 64 ? record_floats(64, true) : D <= 128 ? record_floats(128, true) : D <= 256 ? record_floats(256, true) : 0;
 }
 PBE_EXPORT int pbe_delta_chunk_tokens() { return CH; }
 
@@ -926,7 +641,7 @@ PBE_EXPORT int pbe_delta_scan_chunks(const float* qk, float* v, const float* bet
   if ((D & 3) == 0 && (((uintptr_t)qk | (per_channel ? (uintptr_t)decay : 0)) & 15) != 0)
     return (int)cudaErrorMisalignedAddress;
   const ChunkParams g{qk, decay, beta, v, records, q_start, q_len, R, G, H, D, E};
-  const ChunkScanParams p{records, v, out, state, q_start, q_len, slots, H, D, E, write_state};
+  const ChunkScanParams<float> p{records, v, H * E, out, state, q_start, q_len, slots, H, D, E, write_state};
   const int n = T / CH + R;
   const bool chan = per_channel != 0;
   if (D <= 64) return launch_chunks<4, 2, 4>(g, p, n, chan, stream);

@@ -450,10 +450,11 @@ PBE_EXPORT int pbe_fold_pair(const float* residual, const void* delta_a, const v
 // ---------------------------------------------------------------- gated activations other than silu(g) * u
 // in: [rows, 2*inter], gate in columns [0, inter), linear part in [inter, 2*inter); out [rows, inter].
 // kind 1 (capped swish): g <- min(g, limit), u <- clamp(u, -limit, limit), y = g * sigmoid(alpha * g) * (u + 1).
-// kind 2 (gelu, tanh form): y = gelu_tanh(g) * u.
+// kind 2 (gelu, tanh form): y = gelu_tanh(g) * u.  kind 3 (relu): y = max(g, 0) * u.
+// bias (float32 [2*inter], optional) is added to both first.
 template <typename T>
-__global__ void glu_act_kernel(const T* __restrict__ in, T* __restrict__ out, int inter, size_t total, int kind,
-                               float limit, float alpha) {
+__global__ void glu_act_kernel(const T* __restrict__ in, const float* __restrict__ bias, T* __restrict__ out, int inter,
+                               size_t total, int kind, float limit, float alpha) {
   pdl_launch_dependents();
   pdl_wait();
   for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total;
@@ -462,8 +463,14 @@ __global__ void glu_act_kernel(const T* __restrict__ in, T* __restrict__ out, in
     const int c = (int)(idx - r * inter);
     float g = to_float(in[r * 2 * inter + c]);
     float u = to_float(in[r * 2 * inter + inter + c]);
+    if (bias) {
+      g += bias[c];
+      u += bias[inter + c];
+    }
     float y;
-    if (kind == 1) {
+    if (kind == 3) {
+      y = fmaxf(g, 0.f) * u;
+    } else if (kind == 1) {
       g = fminf(g, limit);
       u = fminf(fmaxf(u, -limit), limit);
       y = (g / (1.0f + expf(-alpha * g))) * (u + 1.0f);
@@ -532,13 +539,52 @@ __global__ void gelu_mul_bf16x8_kernel(const __nv_bfloat16* __restrict__ in, __n
   }
 }
 
-PBE_EXPORT int pbe_glu_act(const void* in, void* out, int dtype, int rows, int inter, int kind, float limit,
-                           float alpha, cudaStream_t stream) {
+// max(g, 0) * u on bfloat16 rows with optional biases, eight values a thread
+__global__ void relu_mul_bf16x8_kernel(const __nv_bfloat16* __restrict__ in, const float* __restrict__ bias,
+                                       __nv_bfloat16* __restrict__ out, int inter, int rows) {
+  pdl_launch_dependents();
+  const int chunk = blockIdx.x * blockDim.x + threadIdx.x;
+  float bg[8], bu[8];
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    const bool have = bias != nullptr && chunk * 8 < inter;
+    bg[i] = have ? bias[chunk * 8 + i] : 0.f;
+    bu[i] = have ? bias[inter + chunk * 8 + i] : 0.f;
+  }
+  pdl_wait();
+  if (chunk * 8 >= inter) return;
+  for (int r = blockIdx.y; r < rows; r += gridDim.y) {
+    const __nv_bfloat16* row = in + (size_t)r * 2 * inter;
+    const uint4 gq = *reinterpret_cast<const uint4*>(row + chunk * 8);
+    const uint4 uq = *reinterpret_cast<const uint4*>(row + inter + chunk * 8);
+    const unsigned gw[4] = {gq.x, gq.y, gq.z, gq.w}, uw[4] = {uq.x, uq.y, uq.z, uq.w};
+    unsigned yw[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float2 g = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gw[i]));
+      const float2 u = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&uw[i]));
+      const __nv_bfloat162 y = __floats2bfloat162_rn(fmaxf(g.x + bg[2 * i], 0.f) * (u.x + bu[2 * i]),
+                                                     fmaxf(g.y + bg[2 * i + 1], 0.f) * (u.y + bu[2 * i + 1]));
+      yw[i] = *reinterpret_cast<const unsigned*>(&y);
+    }
+    *reinterpret_cast<uint4*>(out + (size_t)r * inter + chunk * 8) = make_uint4(yw[0], yw[1], yw[2], yw[3]);
+  }
+}
+
+PBE_EXPORT int pbe_glu_act(const void* in, const float* bias, void* out, int dtype, int rows, int inter, int kind,
+                           float limit, float alpha, cudaStream_t stream) {
   const size_t total = (size_t)rows * inter;
   if (total == 0) return 0;
-  if (kind != 0 && dtype == PBE_BF16 && (inter & 7) == 0 && (((uintptr_t)in | (uintptr_t)out) & 15) == 0) {
+  if (kind != 0 && (kind == 3 || !bias) && dtype == PBE_BF16 && (inter & 7) == 0 &&
+      (((uintptr_t)in | (uintptr_t)out) & 15) == 0) {
     const int threads = 256, chunks = inter / 8;
     dim3 grid((chunks + threads - 1) / threads, rows < 65535 ? rows : 65535);
+    if (kind == 3) {
+      if (grid.y > 512) grid.y = 512;          // a block keeps its biases over several rows
+      launch_k(relu_mul_bf16x8_kernel, grid, threads, 0, stream, (const __nv_bfloat16*)in, bias, (__nv_bfloat16*)out,
+               inter, rows);
+      return launch_status();
+    }
     if (kind == 2) {
       launch_k(gelu_mul_bf16x8_kernel, grid, threads, 0, stream, (const __nv_bfloat16*)in, (__nv_bfloat16*)out, inter,
                rows);
@@ -551,10 +597,10 @@ PBE_EXPORT int pbe_glu_act(const void* in, void* out, int dtype, int rows, int i
   size_t blocks = (total + 255) / 256;
   if (blocks > 148 * 16) blocks = 148 * 16;
   if (dtype == PBE_F32)
-    launch_k(glu_act_kernel<float>, (int)blocks, 256, 0, stream, (const float*)in, (float*)out, inter, total, kind,
+    launch_k(glu_act_kernel<float>, (int)blocks, 256, 0, stream, (const float*)in, bias, (float*)out, inter, total, kind,
              limit, alpha);
   else
-    launch_k(glu_act_kernel<__nv_bfloat16>, (int)blocks, 256, 0, stream, (const __nv_bfloat16*)in,
+    launch_k(glu_act_kernel<__nv_bfloat16>, (int)blocks, 256, 0, stream, (const __nv_bfloat16*)in, bias,
              (__nv_bfloat16*)out, inter, total, kind, limit, alpha);
   return launch_status();
 }

@@ -33,11 +33,11 @@ namespace cg = cooperative_groups;
 struct SkinnyParams {
   const bf16* X;      // [M, K]
   const bf16* W;      // [N, K]
-  const float* bias;  // [N] or null (plain epilogue)
+  const float* bias;  // [N] or null
   void* Y;            // [M, N_out]
   int M, N, K;
   int n_out;          // row stride of Y: N (plain) or N / 2 (SwiGLU)
-  int glu;            // the gated epilogue's activation: 0 silu, 1 gelu (tanh form)
+  int glu;            // the gated epilogue's activation: 0 silu, 1 gelu (tanh form), 2 relu; the plain one's: 3 relu squared
   int tiles;          // 16-row tiles (plain: ceil(N/16); SwiGLU: ceil((N/2)/8))
 };
 
@@ -242,18 +242,25 @@ gemm_skinny_kernel(SkinnyParams p) {
       if (m >= p.M) continue;
       if (SWIGLU) {
         if (row_a < 0) continue;
-        const float gate = acc[nt][j], up = acc[nt][2 + j];
-        const float act = p.glu ? gelu_tanh(gate) : gate * (1.0f / (1.0f + expf(-gate)));
+        float gate = acc[nt][j], up = acc[nt][2 + j];
+        if (p.bias) {
+          gate += p.bias[row_a];
+          up += p.bias[row_b];
+        }
+        const float act = p.glu == 2 ? fmaxf(gate, 0.f)
+                          : p.glu ? gelu_tanh(gate) : gate * (1.0f / (1.0f + expf(-gate)));
         Y[(size_t)m * p.n_out + row_a] = from_float<TY>(act * up);
       } else {
         if (row_a >= 0) {
           float v = acc[nt][j];
           if (p.bias) v += p.bias[row_a];
+          if (p.glu == 3) v = fmaxf(v, 0.f) * fmaxf(v, 0.f);
           Y[(size_t)m * p.n_out + row_a] = from_float<TY>(v);
         }
         if (row_b >= 0) {
           float v = acc[nt][2 + j];
           if (p.bias) v += p.bias[row_b];
+          if (p.glu == 3) v = fmaxf(v, 0.f) * fmaxf(v, 0.f);
           Y[(size_t)m * p.n_out + row_b] = from_float<TY>(v);
         }
       }
@@ -290,14 +297,16 @@ int launch(const SkinnyParams& p, cudaStream_t stream) {
 
 PBE_EXPORT int pbe_gemm_skinny_max_rows() { return 16; }
 
-// mode 0: plain; 1: SwiGLU over a [gate; up] weight (N even, Y is [M, N/2]); 3: the same with gelu (tanh form).
+// mode 0: plain; 1: SwiGLU over a [gate; up] weight (N even, Y is [M, N/2]); 3: the same with gelu (tanh form);
+// 5: with relu; 4: plain, the result's relu squared.
 PBE_EXPORT int pbe_gemm_skinny(const void* X, const void* W, const float* bias, void* Y, int y_dtype,
                                int M, int N, int K, int mode, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (M > 16 || K <= 0 || (K & 7) != 0) return (int)cudaErrorInvalidValue;
-  const int glu = mode == 3 ? 1 : 0;
-  if (mode == 3) mode = 1;
-  if (mode == 1 && ((N & 1) || bias != nullptr)) return (int)cudaErrorInvalidValue;
+  const int glu = mode == 3 ? 1 : mode == 5 ? 2 : mode == 4 ? 3 : 0;
+  if (mode == 3 || mode == 5) mode = 1;
+  if (mode == 4) mode = 0;
+  if (mode == 1 && (N & 1)) return (int)cudaErrorInvalidValue;
   SkinnyParams p;
   p.glu = glu;
   p.X = (const bf16*)X;

@@ -12,7 +12,7 @@
 // read as they lie.  A may be float32 (rounded to bfloat16 as it is staged).  Sums run over K in
 // one fixed order, so a row's result does not depend on the other rows.
 //
-// Epilogues of the heads form: a sigmoid gate per (row, group), and a tail of `rot` values copied
+// Epilogues: relu squared; of the heads form also a sigmoid gate per (row, group), and a tail of `rot` values copied
 // from behind A's K columns to behind the output's N columns, rotated by the rows' positions
 // (pairs (2i, 2i + 1) of its first rot_dims values).
 #include "common.cuh"
@@ -42,6 +42,7 @@ struct GroupGemmParams {
   const int32_t* positions;
   float rot_scale;           // cos and sin of the tail's rotation are both multiplied by it
   int gate_each;             // the gate has a value per output column: gate[t * ldg + g * N + n]
+  int act;                   // 1: the result's relu squared
 };
 
 __device__ __forceinline__ void mma16816(float (&c)[4], const unsigned (&a)[4], unsigned b0, unsigned b1) {
@@ -208,8 +209,13 @@ __global__ void __launch_bounds__(128) grouped_gemm_kernel(GroupGemmParams p) {
           if (n < p.N) g0 = 1.0f / (1.0f + expf(-__bfloat162float(gates[n])));
           if (n + 1 < p.N) g1 = 1.0f / (1.0f + expf(-__bfloat162float(gates[n + 1])));
         }
-        if (n < p.N) out[(size_t)t * p.ldo + n] = from_float<TO>(acc[i][j][2 * hh] * g0);
-        if (n + 1 < p.N) out[(size_t)t * p.ldo + n + 1] = from_float<TO>(acc[i][j][2 * hh + 1] * g1);
+        float y0 = acc[i][j][2 * hh], y1 = acc[i][j][2 * hh + 1];
+        if (p.act == 1) {
+          y0 = fmaxf(y0, 0.f) * fmaxf(y0, 0.f);
+          y1 = fmaxf(y1, 0.f) * fmaxf(y1, 0.f);
+        }
+        if (n < p.N) out[(size_t)t * p.ldo + n] = from_float<TO>(y0 * g0);
+        if (n + 1 < p.N) out[(size_t)t * p.ldo + n + 1] = from_float<TO>(y1 * g1);
       }
     }
   if (p.rot > 0 && blockIdx.z == 0) {
@@ -266,11 +272,11 @@ PBE_EXPORT int pbe_grouped_gemm(const void* a, int a_dtype, int lda, long long a
                                 int wk, int wn, void* out, int out_dtype, int ldo, long long out_group, int T, int K,
                                 int N, int groups, const int32_t* tiles, int num_tiles, const void* gate, int ldg,
                                 int rot, int rot_dims, const float* inv_freq, const int32_t* positions,
-                                float rot_scale, int gate_each, cudaStream_t stream) {
+                                float rot_scale, int gate_each, int act, cudaStream_t stream) {
   if (groups <= 0 || (tiles == nullptr && T <= 0) || (tiles != nullptr && num_tiles <= 0)) return 0;
   GroupGemmParams p{a, lda, a_group, (const __nv_bfloat16*)w, w_group, wk, wn, out, ldo, out_group, T, K, N, groups,
                     tiles, (const __nv_bfloat16*)gate, ldg, rot, rot_dims, inv_freq, positions, rot_scale,
-                    gate_each};
+                    gate_each, act};
   int nz = (N + GG_BN - 1) / GG_BN;
   if (nz == 0) nz = 1;
   dim3 grid = tiles ? dim3(num_tiles, 1, nz) : dim3((T + GG_BM - 1) / GG_BM, groups, nz);

@@ -19,6 +19,10 @@
 //   values into the pages.  The angle's fraction of a turn is formed from the frequency as two
 //   float32 numbers and the exact remainder of the product, so it is good to a few 1e-8 of a turn at
 //   any position.  cos and sin of the values' angles are left in a table for the attention's epilogue.
+// head_conv_norm_write: the same behind a short causal convolution on every channel of queries, keys and values
+//   (taps inputs per channel: the projection's rows of this step, before them the request's state row).  A warp
+//   a head of a token, V neighbouring channels a lane.  A request that brings one token has its convolution
+//   state moved on in the same launch: each channel is read and written by one thread only.
 // masked_attention: the float32-arithmetic kernel.  It reads the engine's attention work list
 //   (request, row tile, key split, splits): the rows of a request are packed with the query heads
 //   that share a key/value head, 16 packed rows a block, 32 keys a tile (a key a lane), online
@@ -29,6 +33,7 @@
 #include "common.cuh"
 #include "masked_attention.cuh"
 #include "pdl.cuh"
+#include "vec.cuh"
 
 using namespace pbe;
 
@@ -164,6 +169,149 @@ __global__ void __launch_bounds__(128) head_norm_write_kernel(HeadNormParams p) 
       ((T*)p.v_pages)[(((size_t)page * G + head) * PT + off) * E + e] = from_float<T>(y);
     }
   }
+}
+
+// ------------------------------------------------------------------ head_conv_norm_write
+struct HeadConvParams {
+  HeadNormParams b;          // what head_norm_write reads (columns from 0: queries, keys, values side by side; no
+                             // bias, no factor per head, no rotation of values)
+  const float* conv_t;       // [taps, C], C = H D + G D + G E; the last tap is the current token's
+  float* conv_state;         // [slots, taps - 1, C], the newest input last
+  const int32_t* request_of_row;
+  const int32_t* q_start;
+  const int32_t* q_len;
+  const int32_t* state_slots;
+  int R, taps, update;
+};
+
+constexpr int HC_WARPS = 4;
+
+// The convolution of V neighbouring channels from column c of one token.
+template <typename T, int V>
+__device__ __forceinline__ void conv_at(const HeadConvParams& p, int t, int i, const float* st_in, float* st_out, int C,
+                                        int c, float (&acc)[V]) {
+#pragma unroll
+  for (int k = 0; k < V; ++k) acc[k] = 0.f;
+  const int taps = p.taps;
+  const T* in = (const T*)p.b.proj + c;
+#pragma unroll 4
+  for (int j = 0; j < taps; ++j) {
+    const int off = i - (taps - 1) + j;          // the input's place among this step's rows; negative: before them
+    float u[V], w[V];
+    if (off >= 0) load_v<V>(in + (size_t)(t - (taps - 1) + j) * p.b.ld, u);
+    else load_v<V>(st_in + (size_t)(taps - 1 + off) * C + c, u);
+    load_v<V>(p.conv_t + (size_t)j * C + c, w);
+#pragma unroll
+    for (int k = 0; k < V; ++k) acc[k] = fmaf(w[k], u[k], acc[k]);
+    if (st_out && j > 0) put_v<V>(st_out + (size_t)(j - 1) * C + c, u);     // entry j - 1 was read the turn before
+  }
+}
+
+// grid (rows, groups of heads_here heads): queries, keys, then values.  N: groups of 32 V channels a head has at most.
+template <typename T, int V, int N>
+__global__ void __launch_bounds__(HC_WARPS * 32) head_conv_norm_write_kernel(HeadConvParams p, int heads_here) {
+  __shared__ float2 rot_cs[16 * HN_MAX];
+  __shared__ __align__(16) float held[HC_WARPS][32 * HN_MAX];      // a warp's head between the norm and the turn
+  pdl_launch_dependents();
+  pdl_wait();
+  const HeadNormParams& b = p.b;
+  const int t = blockIdx.x;
+  const int H = b.H, G = b.G, D = b.D, E = b.E, PT = b.page_tokens;
+  const int C = (H + G) * D + G * E;
+  const int r = p.request_of_row[t];
+  const bool live = r >= 0 && r < p.R && p.q_len[r] > 0;        // not a padding row of a captured step
+  const int half = b.rot_freq ? b.rot_dims / 2 : 0;
+  if (half) {
+    const int pos = b.positions[t];
+    for (int i = threadIdx.x; i < half; i += blockDim.x) rot_cs[i] = turn_of(pos, b.rot_freq[i]);
+    __syncthreads();
+  }
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int slot = (live && b.slots) ? b.slots[t] : -1;
+  const bool store = slot >= 0 && b.k_pages != nullptr;
+  const int page = store ? slot / PT : 0, off = store ? slot - page * PT : 0;
+  const int i = live ? t - p.q_start[r] : 0;
+  float* st = live && p.taps > 1 ? p.conv_state + (size_t)p.state_slots[r] * (p.taps - 1) * C : nullptr;
+  float* st_out = (live && p.update && p.q_len[r] == 1) ? st : nullptr;
+  const int first = blockIdx.y * heads_here, last = min(H + 2 * G, first + heads_here);
+  for (int hh = first + warp; hh < last; hh += HC_WARPS) {
+    if (hh >= H + G) {                         // a value head
+      const int head = hh - H - G;
+      if (!store && !st_out) continue;
+#pragma unroll
+      for (int n = 0; n < N; ++n) {
+        const int e = (n * 32 + lane) * V;
+        if (e < E && live) {
+          float v[V];
+          conv_at<T, V>(p, t, i, st, st_out, C, (H + G) * D + head * E + e, v);
+          if (store) put_v<V>((T*)b.v_pages + (((size_t)page * G + head) * PT + off) * E + e, v);
+        }
+      }
+      continue;
+    }
+    const bool is_q = hh < H;
+    const int head = is_q ? hh : hh - H;
+    if (!is_q && !store && !st_out) continue;
+    const float* gain = is_q ? b.q_gain : b.k_gain;
+    float x[N][V];
+    float ss = 0.f;
+#pragma unroll
+    for (int n = 0; n < N; ++n) {
+      const int d = (n * 32 + lane) * V;
+#pragma unroll
+      for (int k = 0; k < V; ++k) x[n][k] = 0.f;
+      if (d < D && live) conv_at<T, V>(p, t, i, st, st_out, C, hh * D + d, x[n]);
+#pragma unroll
+      for (int k = 0; k < V; ++k) ss = fmaf(x[n][k], x[n][k], ss);
+    }
+    const float sc = gain ? 1.0f / sqrtf(warp_sum(ss) / (float)D + b.eps) : 1.f;
+    __syncwarp();                              // the warp's head before is read
+#pragma unroll
+    for (int n = 0; n < N; ++n) {
+      const int d = (n * 32 + lane) * V;
+      if (d < D) {
+        if (gain) {
+          float g[V];
+          load_v<V>(gain + d, g);
+#pragma unroll
+          for (int k = 0; k < V; ++k) x[n][k] = (x[n][k] * sc) * g[k];
+        }
+        if (d < 2 * half) put_v<V>(&held[warp][d], x[n]);
+      }
+    }
+    __syncwarp();
+#pragma unroll
+    for (int n = 0; n < N; ++n) {
+      const int d = (n * 32 + lane) * V;
+      if (d >= D) continue;
+#pragma unroll
+      for (int k = 0; k < V; ++k) {
+        const int dd = d + k;
+        if (dd < 2 * half) {
+          const bool lower = dd < half;
+          const float other = held[warp][lower ? dd + half : dd - half];
+          const float2 cs = rot_cs[lower ? dd : dd - half];
+          x[n][k] = lower ? x[n][k] * cs.x - other * cs.y : x[n][k] * cs.x + other * cs.y;
+        }
+      }
+      if (is_q) put_v<V>(b.q_out + ((size_t)t * H + head) * D + d, x[n]);
+      else if (store) put_v<V>((T*)b.k_pages + (((size_t)page * G + head) * PT + off) * D + d, x[n]);
+    }
+  }
+}
+
+template <typename T, int V>
+int launch_head_conv(const HeadConvParams& p, int T_rows, cudaStream_t stream) {
+  const int wide = p.b.D > p.b.E ? p.b.D : p.b.E, heads = p.b.H + 2 * p.b.G;
+  // few rows: a block per group of four heads; many: a block keeps its row's angles for all heads
+  const int here = T_rows >= 512 ? heads : HC_WARPS;
+  dim3 grid(T_rows, (heads + here - 1) / here);
+  const int per = (wide + 32 * V - 1) / (32 * V);
+  if (per <= 1) launch_k(head_conv_norm_write_kernel<T, V, 1>, grid, HC_WARPS * 32, 0, stream, p, here);
+  else if (per <= 2) launch_k(head_conv_norm_write_kernel<T, V, 2>, grid, HC_WARPS * 32, 0, stream, p, here);
+  else if (per <= 8 / V) launch_k(head_conv_norm_write_kernel<T, V, 8 / V>, grid, HC_WARPS * 32, 0, stream, p, here);
+  else return (int)cudaErrorInvalidValue;
+  return launch_status();
 }
 
 // ------------------------------------------------------------------ masked_attention
@@ -515,6 +663,36 @@ PBE_EXPORT int pbe_head_norm_write(const void* proj, int ld, int q_off, int k_of
     else launch_k(head_norm_write_kernel<__nv_bfloat16, false>, T, 128, 0, stream, p);
   }
   return launch_status();
+}
+
+PBE_EXPORT int pbe_head_conv_norm_write(const void* proj, int ld, const float* conv_t, float* conv_state,
+                                        const float* q_gain, const float* k_gain, const int32_t* slots, float* q_out,
+                                        void* k_pages, void* v_pages, int T, int R, int H, int G, int D, int E,
+                                        int page_tokens, float eps, const int32_t* positions, const float2* rot_freq,
+                                        int rot_dims, int taps, int update, const int32_t* request_of_row,
+                                        const int32_t* q_start, const int32_t* q_len, const int32_t* state_slots,
+                                        int dtype, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (D > 32 * HN_MAX || E > 32 * HN_MAX || D < 1 || E < 1 || taps < 1 || taps > 16) return (int)cudaErrorInvalidValue;
+  if (rot_freq && (positions == nullptr || rot_dims < 2 || (rot_dims & 1) || rot_dims > D)) return (int)cudaErrorInvalidValue;
+  HeadConvParams p{};
+  p.b = HeadNormParams{proj, ld, 0, H * D, (H + G) * D, nullptr, q_gain, k_gain, nullptr, slots, q_out, k_pages,
+                       v_pages, H, G, D, E, page_tokens, eps, positions, rot_freq, rot_dims, nullptr, nullptr};
+  p.conv_t = conv_t;
+  p.conv_state = conv_state;
+  p.request_of_row = request_of_row;
+  p.q_start = q_start;
+  p.q_len = q_len;
+  p.state_slots = state_slots;
+  p.R = R;
+  p.taps = taps;
+  p.update = update;
+  const bool f32 = dtype == PBE_F32;
+  const bool vec4 = D % 4 == 0 && E % 4 == 0 && ld % 4 == 0 &&
+                    (((uintptr_t)conv_t | (uintptr_t)conv_state | (uintptr_t)q_out | (uintptr_t)q_gain | (uintptr_t)k_gain) & 15) == 0 &&
+                    (((uintptr_t)proj | (uintptr_t)k_pages | (uintptr_t)v_pages) & (f32 ? 15 : 7)) == 0;
+  if (f32) return vec4 ? launch_head_conv<float, 4>(p, T, stream) : launch_head_conv<float, 1>(p, T, stream);
+  return vec4 ? launch_head_conv<__nv_bfloat16, 4>(p, T, stream) : launch_head_conv<__nv_bfloat16, 1>(p, T, stream);
 }
 
 PBE_EXPORT int pbe_masked_attention(const AttnParams* params, int D, int E, const float* bias, int bias_rows,

@@ -6,8 +6,8 @@
 // 2) the sum of its two largest, and only experts of the `keep` best groups can be chosen (groups =
 // 1: no restriction; a barred expert is out whatever its c, which may be negative); the `top`
 // allowed experts with the largest c are chosen (ties: the lower index); their weights are their
-// scores s, without the correction, over the sum of the chosen scores (+ 1e-20), times `scale`.
-// One warp per token.
+// scores s, without the correction, over the sum of the chosen scores (+ 1e-20) unless they are taken
+// as they are, times `scale`.  One warp per token.
 //
 // expert_rows: for few rows (decoded tokens).  Per (token, chosen expert) pair the expert's gate
 // and up rows are streamed against the token's input (blocks of 32 hidden units, a warp per unit,
@@ -15,6 +15,11 @@
 // a second launch streams the down rows against it (blocks of 32 output columns) and writes the
 // weighted result to the pair's own slot, [T, top, W]; combine adds a token's slots in order, so
 // a token's result never depends on what else is in the step.
+//
+// Experts without a gate (act 2: h = relu(W_up x)^2) have up rows only.  A router's weight may multiply an
+// expert's input instead of its output (weight_in): expert_rows then scales the up product, which is the
+// same, and the gather scales the rows.  What is added for every token (a shared expert) may carry a factor
+// sigmoid(z_t), z one float32 number per token.
 //
 // For many rows the host side sorts the rows by expert (pair_rows / scatter below) and runs one
 // matrix product per expert over its rows.
@@ -28,7 +33,8 @@ constexpr int MAX_PER_LANE = 16;       // experts a lane holds: up to 512 expert
 constexpr int MAX_TOP = 32;
 
 struct RouteParams {
-  const float* logits;       // [T, E]
+  const float* logits;       // [T, ld]
+  int ld;
   int32_t* chosen;           // [T, top]
   float* weights;            // [T, top]
   int T, E, top, groups, keep;
@@ -36,6 +42,7 @@ struct RouteParams {
   int score_kind;            // 0: softmax over the experts, 1: sigmoid
   const float* correction;   // [E] or null: added to the scores for the choice only
   int group_rank;            // 1: a group's largest choice score, 2: the sum of its two largest
+  int normalize;             // 1: the weights are divided by the chosen scores' sum
 };
 
 // the lane-distributed argmax of v (lane l holds experts l, l + 32, ...); ties go to the lower index
@@ -55,7 +62,7 @@ __global__ void route_kernel(RouteParams p) {
   const int t = blockIdx.x * warps + (threadIdx.x >> 5);
   if (t >= p.T) return;
   const int lane = threadIdx.x & 31, E = p.E;
-  const float* z = p.logits + (size_t)t * E;
+  const float* z = p.logits + (size_t)t * p.ld;
   float s[MAX_PER_LANE];     // the scores
   float c[MAX_PER_LANE];     // the choice scores
   if (p.score_kind == 1) {
@@ -182,7 +189,7 @@ __global__ void route_kernel(RouteParams p) {
     total += best_s;
   }
   if (lane == 0) {
-    const float inv = p.scale / (total + 1e-20f);
+    const float inv = p.normalize ? p.scale / (total + 1e-20f) : p.scale;
     for (int k = 0; k < p.top && k < MAX_TOP; ++k) {
       p.chosen[(size_t)t * p.top + k] = picked_e[k];
       p.weights[(size_t)t * p.top + k] = picked_s[k] * inv;
@@ -202,8 +209,10 @@ struct ExpertRowsParams {
   float* hidden;             // [T * top, F] scratch: silu(gate) * up of every pair
   float* part;               // [T, top, W]
   int T, W, F, top;
-  int act;                   // 0: silu(g) * u; 1: g <- min(g, limit), u <- clamp(u, +-limit), g sigmoid(alpha g) (u + 1)
+  int act;                   // 0: silu(g) * u; 1: g <- min(g, limit), u <- clamp(u, +-limit), g sigmoid(alpha g) (u + 1);
+                             // 2: relu(u)^2, no gate
   float limit, alpha;
+  int weight_in;             // 1: the weight multiplies the expert's input
 };
 
 // dot product of a weight row with a float32 vector in shared memory, the lanes along the row;
@@ -259,12 +268,16 @@ __global__ void __launch_bounds__(ER_WARPS * 32) expert_hidden_kernel(ExpertRows
   const T* wg = (const T*)p.w_gate + (size_t)e * p.gu_stride;
   const T* wu = (const T*)p.w_up + (size_t)e * p.gu_stride;
   const int f_end = min(p.F, (blockIdx.y + 1) * ER_UNITS);
+  const float scale_in = p.weight_in ? p.weights[pair] : 1.0f;
   for (int f = blockIdx.y * ER_UNITS + warp; f < f_end; f += ER_WARPS) {
-    const float g = dot_row(wg + (size_t)f * p.W, xs, p.W, lane);
-    const float u = dot_row(wu + (size_t)f * p.W, xs, p.W, lane);
+    const float g = p.act == 2 ? 0.f : dot_row(wg + (size_t)f * p.W, xs, p.W, lane) * scale_in;
+    const float u = dot_row(wu + (size_t)f * p.W, xs, p.W, lane) * scale_in;
     if (lane == 0) {
       float h;
-      if (p.act == 1) {
+      if (p.act == 2) {
+        const float ur = fmaxf(u, 0.f);
+        h = ur * ur;
+      } else if (p.act == 1) {
         const float gc = fminf(g, p.limit), uc = fminf(fmaxf(u, -p.limit), p.limit);
         h = (gc / (1.0f + expf(-p.alpha * gc))) * (uc + 1.0f);
       } else {
@@ -283,7 +296,7 @@ __global__ void __launch_bounds__(ER_WARPS * 32) expert_down_kernel(ExpertRowsPa
   pdl_wait();
   const int pair = blockIdx.x;
   const int e = p.chosen[pair];
-  const float weight = p.weights[pair];
+  const float weight = p.weight_in ? 1.0f : p.weights[pair];
   for (int i = threadIdx.x; i < p.F; i += blockDim.x) hs[i] = p.hidden[(size_t)pair * p.F + i];
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -296,10 +309,16 @@ __global__ void __launch_bounds__(ER_WARPS * 32) expert_down_kernel(ExpertRowsPa
   }
 }
 
-// `addend` (optional, [T, W]): what every token gets besides its experts (a shared expert's output)
+// `addend` (optional, [T, W]): what every token gets besides its experts (a shared expert's output), times
+// sigmoid(gate[t * ld_gate]) when there is a gate
+__device__ __forceinline__ float addend_factor(const float* gate, int ld_gate, size_t t) {
+  return gate ? 1.0f / (1.0f + expf(-gate[t * ld_gate])) : 1.0f;
+}
+
 template <typename T>
-__global__ void combine_kernel(const float* __restrict__ part, const T* __restrict__ addend, T* __restrict__ out,
-                               int top, int W, size_t total) {
+__global__ void combine_kernel(const float* __restrict__ part, const T* __restrict__ addend,
+                               const float* __restrict__ gate, int ld_gate, T* __restrict__ out, int top, int W,
+                               size_t total) {
   pdl_launch_dependents();
   pdl_wait();
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
@@ -307,7 +326,7 @@ __global__ void combine_kernel(const float* __restrict__ part, const T* __restri
     const int c = (int)(i - t * W);
     float a = 0.f;
     for (int k = 0; k < top; ++k) a += part[(t * top + k) * W + c];
-    if (addend) a += to_float(addend[i]);
+    if (addend) a = fmaf(addend_factor(gate, ld_gate, t), to_float(addend[i]), a);
     out[i] = from_float<T>(a);
   }
 }
@@ -350,10 +369,16 @@ __global__ void place_kernel(const int32_t* __restrict__ chosen, int pairs, int 
 template <typename T>
 __global__ void gather_rows_kernel(const T* __restrict__ x, const int32_t* __restrict__ chosen,
                                    const int32_t* __restrict__ place, const int32_t* __restrict__ start,
-                                   T* __restrict__ gathered, int top, int W) {
+                                   const float* __restrict__ weights, T* __restrict__ gathered, int top, int W) {
   const int pair = blockIdx.x;
   const int t = pair / top;
   const size_t dst = (size_t)(start[chosen[pair]] + place[pair]) * W;
+  if (weights) {
+    const float f = weights[pair];
+    for (int i = threadIdx.x; i < W; i += blockDim.x)
+      gathered[dst + i] = from_float<T>(f * to_float(x[(size_t)t * W + i]));
+    return;
+  }
   for (int i = threadIdx.x; i < W; i += blockDim.x) gathered[dst + i] = x[(size_t)t * W + i];
 }
 
@@ -361,29 +386,30 @@ template <typename T>
 __global__ void scatter_rows_kernel(const T* __restrict__ y, const int32_t* __restrict__ chosen,
                                     const int32_t* __restrict__ place, const int32_t* __restrict__ start,
                                     const float* __restrict__ weights, const T* __restrict__ addend,
-                                    T* __restrict__ out, int top, int W) {
+                                    const float* __restrict__ gate, int ld_gate, T* __restrict__ out, int top, int W) {
   const int t = blockIdx.x;
+  const float factor = addend_factor(gate, ld_gate, t);
   for (int i = threadIdx.x; i < W; i += blockDim.x) {
     float a = 0.f;
     for (int k = 0; k < top; ++k) {
       const int pair = t * top + k;
-      a += weights[pair] * to_float(y[(size_t)(start[chosen[pair]] + place[pair]) * W + i]);
+      a += (weights ? weights[pair] : 1.0f) * to_float(y[(size_t)(start[chosen[pair]] + place[pair]) * W + i]);
     }
-    if (addend) a += to_float(addend[(size_t)t * W + i]);
+    if (addend) a = fmaf(factor, to_float(addend[(size_t)t * W + i]), a);
     out[(size_t)t * W + i] = from_float<T>(a);
   }
 }
 }  // namespace
 
-PBE_EXPORT int pbe_route(const float* logits, int32_t* chosen, float* weights, int T, int E, int top, int groups,
+PBE_EXPORT int pbe_route(const float* logits, int ld, int32_t* chosen, float* weights, int T, int E, int top, int groups,
                          int keep, float scale, int score_kind, const float* correction, int group_rank,
-                         cudaStream_t stream) {
+                         int normalize, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (E < 1 || E > 32 * MAX_PER_LANE || top < 1 || top > MAX_TOP || top > E || groups < 1 || groups > 64 ||
       E % groups != 0 || keep < 1 || keep > groups || top > keep * (E / groups) || score_kind < 0 || score_kind > 1 ||
       group_rank < 1 || group_rank > 2)
     return (int)cudaErrorInvalidValue;
-  RouteParams p{logits, chosen, weights, T, E, top, groups, keep, scale, score_kind, correction, group_rank};
+  RouteParams p{logits, ld, chosen, weights, T, E, top, groups, keep, scale, score_kind, correction, group_rank, normalize};
   launch_k(route_kernel, (T + 3) / 4, 128, 0, stream, p);
   return launch_status();
 }
@@ -391,9 +417,10 @@ PBE_EXPORT int pbe_route(const float* logits, int32_t* chosen, float* weights, i
 PBE_EXPORT int pbe_expert_rows(const void* x, const void* w_gate, const void* w_up, long long gu_stride,
                                const void* w_down, const int32_t* chosen, const float* weights, float* hidden,
                                float* part, void* out, int dtype, int T, int W, int F, int top, int act, float limit,
-                               float alpha, const void* addend, cudaStream_t stream) {
+                               float alpha, const void* addend, const float* addend_gate, int ld_gate, int weight_in,
+                               cudaStream_t stream) {
   if (T <= 0) return 0;
-  ExpertRowsParams p{x, w_gate, w_up, gu_stride, w_down, chosen, weights, hidden, part, T, W, F, top, act, limit, alpha};
+  ExpertRowsParams p{x, w_gate, w_up, gu_stride, w_down, chosen, weights, hidden, part, T, W, F, top, act, limit, alpha, weight_in};
   const size_t smem1 = sizeof(float) * (size_t)W, smem2 = sizeof(float) * (size_t)F;
   if (smem1 > 200 * 1024 || smem2 > 200 * 1024) return (int)cudaErrorInvalidValue;
   dim3 grid1(T * top, (F + ER_UNITS - 1) / ER_UNITS), grid2(T * top, (W + ER_UNITS - 1) / ER_UNITS);
@@ -416,11 +443,11 @@ PBE_EXPORT int pbe_expert_rows(const void* x, const void* w_gate, const void* w_
   size_t blocks = (total + 255) / 256;
   if (blocks > 148 * 16) blocks = 148 * 16;
   if (dtype == PBE_F32)
-    launch_k(combine_kernel<float>, (int)blocks, 256, 0, stream, (const float*)part, (const float*)addend, (float*)out,
-             top, W, total);
+    launch_k(combine_kernel<float>, (int)blocks, 256, 0, stream, (const float*)part, (const float*)addend, addend_gate,
+             ld_gate, (float*)out, top, W, total);
   else
     launch_k(combine_kernel<__nv_bfloat16>, (int)blocks, 256, 0, stream, (const float*)part,
-             (const __nv_bfloat16*)addend, (__nv_bfloat16*)out, top, W, total);
+             (const __nv_bfloat16*)addend, addend_gate, ld_gate, (__nv_bfloat16*)out, top, W, total);
   return launch_status();
 }
 
@@ -432,25 +459,27 @@ PBE_EXPORT int pbe_expert_places(const int32_t* chosen, int pairs, int E, int32_
 }
 
 PBE_EXPORT int pbe_expert_gather(const void* x, const int32_t* chosen, const int32_t* place, const int32_t* start,
-                                 void* gathered, int dtype, int T, int top, int W, cudaStream_t stream) {
+                                 const float* weights, void* gathered, int dtype, int T, int top, int W,
+                                 cudaStream_t stream) {
   if (T <= 0) return 0;
   if (dtype == PBE_F32)
-    gather_rows_kernel<float><<<T * top, 128, 0, stream>>>((const float*)x, chosen, place, start, (float*)gathered, top, W);
+    gather_rows_kernel<float><<<T * top, 128, 0, stream>>>((const float*)x, chosen, place, start, weights, (float*)gathered, top, W);
   else
-    gather_rows_kernel<__nv_bfloat16><<<T * top, 128, 0, stream>>>((const __nv_bfloat16*)x, chosen, place, start,
+    gather_rows_kernel<__nv_bfloat16><<<T * top, 128, 0, stream>>>((const __nv_bfloat16*)x, chosen, place, start, weights,
                                                                   (__nv_bfloat16*)gathered, top, W);
   return launch_status();
 }
 
 PBE_EXPORT int pbe_expert_scatter(const void* y, const int32_t* chosen, const int32_t* place, const int32_t* start,
                                   const float* weights, void* out, int dtype, int T, int top, int W,
-                                  const void* addend, cudaStream_t stream) {
+                                  const void* addend, const float* addend_gate, int ld_gate, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (dtype == PBE_F32)
     scatter_rows_kernel<float><<<T, 128, 0, stream>>>((const float*)y, chosen, place, start, weights,
-                                                     (const float*)addend, (float*)out, top, W);
+                                                     (const float*)addend, addend_gate, ld_gate, (float*)out, top, W);
   else
     scatter_rows_kernel<__nv_bfloat16><<<T, 128, 0, stream>>>((const __nv_bfloat16*)y, chosen, place, start, weights,
-                                                             (const __nv_bfloat16*)addend, (__nv_bfloat16*)out, top, W);
+                                                             (const __nv_bfloat16*)addend, addend_gate, ld_gate,
+                                                             (__nv_bfloat16*)out, top, W);
   return launch_status();
 }

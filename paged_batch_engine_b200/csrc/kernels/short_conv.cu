@@ -33,6 +33,7 @@ struct ConvParams {
   const int32_t* slots;      // [R] state row of each request
   int T, R, C, taps;
   int act;                   // 1: silu
+  int skip = 0;              // the state of requests of at most this many tokens stays as it is
 };
 
 template <typename T>
@@ -127,7 +128,7 @@ __global__ void short_conv_state_kernel(ConvParams p) {
   const int c = blockIdx.y * blockDim.x + threadIdx.x;
   if (c >= p.C) return;
   const int n = p.q_len[r];
-  if (n <= 0) return;
+  if (n <= p.skip) return;
   const int keep = p.taps - 1;
   float* st = p.state + (size_t)p.slots[r] * keep * p.C + c;
   const T* in = (const T*)p.in + c;
@@ -194,6 +195,20 @@ PBE_EXPORT int pbe_short_conv(const void* in, int ld, int dtype, const float* we
   dim3 grid2(R, (C + threads - 1) / threads);
   if (dtype == PBE_F32) launch_k(short_conv_state_kernel<float>, grid2, threads, 0, stream, p);
   else launch_k(short_conv_state_kernel<__nv_bfloat16>, grid2, threads, 0, stream, p);
+  return launch_status();
+}
+
+// The state alone, for a caller that convolved by itself: moved on for requests of more than `skip` tokens.
+PBE_EXPORT int pbe_conv_state(const void* in, int ld, int dtype, float* state, const int32_t* q_start,
+                              const int32_t* q_len, const int32_t* slots, int R, int C, int taps, int skip,
+                              cudaStream_t stream) {
+  if (R <= 0 || C <= 0 || taps == 1) return 0;
+  if (taps < 1 || taps > MAX_TAPS) return (int)cudaErrorInvalidValue;
+  ConvParams p{in, ld, nullptr, nullptr, nullptr, state, nullptr, nullptr, q_start, q_len, slots, 0, R, C, taps, 0, skip};
+  const int threads = C >= 256 ? 256 : 128;
+  dim3 grid(R, (C + threads - 1) / threads);
+  if (dtype == PBE_F32) launch_k(short_conv_state_kernel<float>, grid, threads, 0, stream, p);
+  else launch_k(short_conv_state_kernel<__nv_bfloat16>, grid, threads, 0, stream, p);
   return launch_status();
 }
 

@@ -136,7 +136,7 @@ def block_desc(block) -> Optional[BlockDesc]:
         getattr(block, "norm2", None)
     if not (type(m) is GQAttention and type(f) is SwiGLU and type(n1) is RMSNorm and type(n2) is RMSNorm):
         return None
-    if f.activation != "silu" or n1.on_output or n2.on_output:
+    if f.activation != "silu" or f.bias or n1.on_output or n2.on_output:
         return None
     if m.dtype != torch.bfloat16 or m.o_bias or m.kernel_kind == "simple":
         return None

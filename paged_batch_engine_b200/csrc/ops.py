@@ -158,24 +158,30 @@ def fold_pair(residual: torch.Tensor, delta_a: Optional[torch.Tensor], delta_b: 
     return out
 
 
-GLU_ACTIVATIONS = {"silu": 0, "capped_swish": 1, "gelu_tanh": 2}
-GLU_EPILOGUES = {"silu": 1, "gelu_tanh": 3}      # those the few-row products have as an epilogue, and their mode
+GLU_ACTIVATIONS = {"silu": 0, "capped_swish": 1, "gelu_tanh": 2, "relu": 3}
+# the gated activations the few-row products have as an epilogue, and their mode there
+SKINNY_GLU = {"silu": 1, "gelu_tanh": 3, "relu": 5}
+STREAM_GLU = {"silu": 1, "gelu_tanh": 3}
+UNGATED_EXPERTS = {"relu2": 2}      # expert activations without a gate, and their code in the expert kernels
 
 
 def gated_activation(gate_up: torch.Tensor, out: torch.Tensor, activation: str = "silu", limit: float = 0.0,
-                     alpha: float = 1.0) -> torch.Tensor:
+                     alpha: float = 1.0, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """out[r, c] = act(gate_up[r, c], gate_up[r, inter + c]).  "silu": silu(g) * u.  "capped_swish":
     g <- min(g, limit), u <- clamp(u, -limit, limit), g * sigmoid(alpha * g) * (u + 1).  "gelu_tanh": gelu(g) * u in
-    gelu's tanh form."""
-    if activation == "silu":
+    gelu's tanh form.  "relu": max(g, 0) * u.  ``bias`` (float32 [2 * inter]) is added to both first."""
+    if activation == "silu" and bias is None:
         return silu_mul(gate_up, out)
-    _need_cuda(gate_up, out)
-    _need_contiguous(gate_up, out)
+    _need_cuda(gate_up, out, bias)
+    _need_contiguous(gate_up, out, bias)
     rows, two_i = gate_up.shape
     if two_i % 2 or out.shape != (rows, two_i // 2) or out.dtype != gate_up.dtype:
         raise KernelError("gated_activation: shapes or dtypes do not agree")
-    fn = _fn("elementwise", "pbe_glu_act", [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p])
-    _check(fn(_ptr(gate_up), _ptr(out), _dtype_code(out), rows, two_i // 2, GLU_ACTIVATIONS[activation], float(limit),
+    if bias is not None and (bias.dtype != torch.float32 or bias.numel() != two_i):
+        raise KernelError("gated_activation: the bias is float32 [2 * inter]")
+    fn = _fn("elementwise", "pbe_glu_act", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float,
+                                            c_void_p])
+    _check(fn(_ptr(gate_up), _ptr(bias), _ptr(out), _dtype_code(out), rows, two_i // 2, GLU_ACTIVATIONS[activation], float(limit),
               float(alpha), _stream()), "gated_activation")
     return out
 
@@ -226,6 +232,33 @@ def norm_add(x: torch.Tensor, y: torch.Tensor, gain: torch.Tensor, eps: float,
     fn = _fn("norm_add", "pbe_norm_add", [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p])
     _check(fn(_ptr(x), _ptr(y), _dtype_code(y), _ptr(gain), _ptr(lp), T, d, float(eps), _stream()), "norm_add")
     return lp
+
+
+def norm_add_norm(x: torch.Tensor, y1: torch.Tensor, y2: Optional[torch.Tensor], scale_1: float, scale_2: float,
+                  gain_b: torch.Tensor, eps_b: float, gain: torch.Tensor, eps: float,
+                  rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """x += gain_b * y / sqrt(mean(y^2) + eps_b) with y = scale_1 y1 + scale_2 y2 (``y2`` optional), in place (x
+    float32 [T, W]), and the norm gain * x / sqrt(mean(x^2) + eps) of the sum, returned in y1's dtype.  With
+    ``rows`` (int32 [n]) output row i is made from batch row rows[i] and x is not written."""
+    _need_cuda(x, y1, y2, gain_b, gain, rows)
+    _need_contiguous(x, y1, y2, gain_b, gain, rows)
+    if x.dtype != torch.float32 or x.dim() != 2 or y1.shape != x.shape:
+        raise KernelError("norm_add_norm: x is float32 [T, W] and y has its shape")
+    if y2 is not None and (y2.shape != y1.shape or y2.dtype != y1.dtype):
+        raise KernelError("norm_add_norm: the two branches agree in shape and dtype")
+    T, d = x.shape
+    for g in (gain_b, gain):
+        if g.dtype != torch.float32 or g.numel() != d:
+            raise KernelError("norm_add_norm: gains are float32 [W]")
+    if rows is not None and rows.dtype != torch.int32:
+        raise KernelError("norm_add_norm: rows are int32")
+    n = T if rows is None else rows.numel()
+    out = torch.empty((n, d), dtype=y1.dtype, device=x.device)
+    fn = _fn("norm_add", "pbe_norm_add_norm", [c_void_p, c_void_p, c_void_p, c_float, c_float, c_int, c_void_p, c_float,
+                                               c_void_p, c_float, c_void_p, c_void_p, c_int, c_int, c_void_p])
+    _check(fn(_ptr(x), _ptr(y1), _ptr(y2), float(scale_1), float(scale_2), _dtype_code(y1), _ptr(gain_b), float(eps_b),
+              _ptr(gain), float(eps), _ptr(out), _ptr(rows), n, d, _stream()), "norm_add_norm")
+    return out
 
 
 def silu_mul(gate_up: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
@@ -611,10 +644,10 @@ SKINNY_MAX_ROWS = int(os.environ.get('PBE_SKINNY_ROWS', '8'))      # batches of 
 
 def gemm_skinny(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
                 out_dtype: Optional[torch.dtype] = None, swiglu: bool = False,
-                activation: str = "silu") -> torch.Tensor:
+                activation: Optional[str] = "silu") -> torch.Tensor:
     """y = x w^T (+ b) for at most 16 rows, bfloat16 operands, weights streamed once.
-    ``swiglu``: w is [gate; up] stacked and y = act(x gate^T) * (x up^T), [M, N/2], with ``activation``
-    one of ``GLU_EPILOGUES``."""
+    ``swiglu``: w is [gate; up] stacked and y = act(x gate^T + b_g) * (x up^T + b_u), [M, N/2], with
+    ``activation`` one of ``SKINNY_GLU``.  Otherwise ``activation`` "relu2" squares the result's relu."""
     _need_cuda(x, w, bias)
     _need_contiguous(x, w, bias)
     M, K = x.shape
@@ -623,8 +656,8 @@ def gemm_skinny(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] =
         raise KernelError("gemm_skinny takes bfloat16 x [M, K] and w [N, K]")
     if M > 16 or K % 8 != 0:
         raise KernelError(f"gemm_skinny takes at most 16 rows and K a multiple of 8 (got M={M}, K={K})")
-    if swiglu and (N % 2 or bias is not None):
-        raise KernelError("gemm_skinny: the SwiGLU epilogue needs an even N and no bias")
+    if swiglu and N % 2:
+        raise KernelError("gemm_skinny: the SwiGLU epilogue needs an even N")
     if bias is not None and (bias.dtype != torch.float32 or bias.numel() != N):
         raise KernelError("gemm_skinny: bias must be float32 [N]")
     out_dtype = out_dtype or torch.bfloat16
@@ -632,7 +665,7 @@ def gemm_skinny(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] =
     fn = _fn("gemm_skinny", "pbe_gemm_skinny",
              [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p])
     _check(fn(_ptr(x), _ptr(w), _ptr(bias), _ptr(out), _dtype_code(out), M, N, K,
-              GLU_EPILOGUES[activation] if swiglu else 0, _stream()), "gemm_skinny")
+              SKINNY_GLU[activation] if swiglu else (4 if activation == "relu2" else 0), _stream()), "gemm_skinny")
     return out
 
 
@@ -683,7 +716,7 @@ def gemm_stream(x: torch.Tensor, w: torch.Tensor, out_dtype: Optional[torch.dtyp
     """y = x w^T for up to 64 rows on the tcgen05 tensor cores with the weights as the streamed
     operand (TMA-fed ring, accumulator in tensor memory, K split over blocks where the matrix has
     few rows).  ``swiglu``: w is [gate; up] stacked and y = act(x gate^T) * (x up^T), [M, N/2], with
-    ``activation`` one of ``GLU_EPILOGUES``.  ``check`` synchronises and raises if a bounded wait inside the kernel ran out."""
+    ``activation`` one of ``STREAM_GLU``.  ``check`` synchronises and raises if a bounded wait inside the kernel ran out."""
     _need_cuda(x, w)
     _need_contiguous(x, w)
     M, K = x.shape
@@ -699,7 +732,7 @@ def gemm_stream(x: torch.Tensor, w: torch.Tensor, out_dtype: Optional[torch.dtyp
     scratch, tickets, err = gemm_stream_buffers(x.device)
     fn = _fn("gemm_stream", "pbe_gemm_stream",
              [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p])
-    _check(fn(_ptr(x), _ptr(w), _ptr(out), _dtype_code(out), M, N, K, GLU_EPILOGUES[activation] if swiglu else 0,
+    _check(fn(_ptr(x), _ptr(w), _ptr(out), _dtype_code(out), M, N, K, STREAM_GLU[activation] if swiglu else 0,
               _ptr(scratch), _ptr(tickets), _ptr(err), _stream()), "gemm_stream")
     if check and int(err.item()) != 0:
         err.zero_()
@@ -822,11 +855,10 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
         return gemm_tc5(x, w, out_dtype)
     if out_dtype == torch.float32:
         y = torch.mm(x, w.t(), out_dtype=torch.float32)
-    else:
-        y = torch.mm(x, w.t())
+        return y if bias is None else y.add_(bias)
     if bias is not None:
-        y += bias.to(y.dtype)
-    return y
+        return torch.addmm(bias.to(x.dtype), x, w.t())
+    return torch.mm(x, w.t())
 
 
 # ------------------------------------------------------------------ attention
@@ -1314,6 +1346,20 @@ def short_conv(u: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tenso
     return out
 
 
+def conv_state_advance(u: torch.Tensor, state: torch.Tensor, q_start: torch.Tensor, q_len: torch.Tensor,
+                       slots: torch.Tensor, num_requests: int, skip: int = 0) -> None:
+    """The convolution state moved on by the rows ``u`` [T, C] (a column slice) of each request that brings more
+    than ``skip`` of them: ``state`` float32 [slots, taps - 1, C], the newest input last."""
+    _need_cuda(u, state, q_start, q_len, slots)
+    _column_slice(u, "conv_state_advance")
+    T, C = u.shape
+    if state.dtype != torch.float32 or state.shape[2] != C or not state.is_contiguous():
+        raise KernelError("conv_state_advance: the state is float32 [slots, taps - 1, C]")
+    fn = _fn("short_conv", "pbe_conv_state", [c_void_p, c_int, c_int] + [c_void_p] * 4 + [c_int] * 4 + [c_void_p])
+    _check(fn(_ptr(u), u.stride(0) if T > 1 else max(u.stride(0), C), _dtype_code(u), _ptr(state), _ptr(q_start), _ptr(q_len),
+              _ptr(slots), int(num_requests), C, state.shape[1] + 1, int(skip), _stream()), "conv_state")
+
+
 def step_sizes(u: torch.Tensor, bias: torch.Tensor, rate_log: torch.Tensor):
     """(dt, decay), float32 [T, H]: dt = softplus(u + bias_h), decay = exp(-exp(rate_log_h) * dt);
     ``u`` [T, H] is a column slice of a projection."""
@@ -1550,11 +1596,73 @@ def head_norm_write(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, bias
     return q if turn is None else (q, turn)
 
 
-def turn_frequencies(pairs: int, base: float, device) -> torch.Tensor:
+def head_conv_norm_write(proj: torch.Tensor, conv_t: torch.Tensor, conv_state: torch.Tensor,
+                         q_gain: Optional[torch.Tensor], k_gain: Optional[torch.Tensor], slots: Optional[torch.Tensor],
+                         k_pages: Optional[torch.Tensor], v_pages: Optional[torch.Tensor], num_heads: int,
+                         num_kv_heads: int, key_dim: int, value_dim: int, page_tokens: int, eps: float,
+                         request_of_row: torch.Tensor, q_start: torch.Tensor, q_len: torch.Tensor,
+                         state_slots: torch.Tensor, num_requests: int, positions: Optional[torch.Tensor] = None,
+                         rot_freq: Optional[torch.Tensor] = None, update_state: bool = True,
+                         single_tokens: bool = False) -> torch.Tensor:
+    """``head_norm_write`` behind a causal convolution on every channel of [q | k | v], the columns the
+    projection [T, ld] begins with: ``conv_t`` float32 [taps, C] (the last tap on the current token),
+    ``conv_state`` float32 [slots, taps - 1, C] with each request's last inputs, read and moved on
+    (``update_state``).  Then the norms, the rotation and the cache write.  ``single_tokens``: every request
+    of the step brings one token.  Returns the queries, float32 [T, H * D]."""
+    H, G, D, E = num_heads, num_kv_heads, key_dim, value_dim
+    _need_cuda(proj, conv_t, conv_state, q_gain, k_gain, slots, k_pages, v_pages, request_of_row, q_start, q_len,
+               state_slots, positions, rot_freq)
+    _need_contiguous(conv_t, conv_state, q_gain, k_gain, slots, k_pages, v_pages, positions, rot_freq)
+    T, C, taps = proj.shape[0], (H + G) * D + G * E, conv_t.shape[0]
+    if proj.dim() != 2 or proj.stride(1) != 1 or proj.shape[1] < C:
+        raise KernelError("head_conv_norm_write: the projection is [T, >= H D + G D + G E] with unit column stride")
+    if conv_t.dtype != torch.float32 or conv_t.shape[1] != C or not 1 <= taps <= 16 or \
+            conv_state.dtype != torch.float32 or tuple(conv_state.shape[1:]) != (taps - 1, C):
+        raise KernelError("head_conv_norm_write: conv_t is float32 [taps, C], the state float32 [slots, taps - 1, C]")
+    for g in (q_gain, k_gain):
+        if g is not None and (g.dtype != torch.float32 or g.numel() != D):
+            raise KernelError("head_conv_norm_write: gains are float32 [key_dim]")
+    if rot_freq is not None and (rot_freq.dtype != torch.float32 or rot_freq.shape[1] != 2 or 2 * rot_freq.shape[0] > D
+                                 or positions is None or positions.dtype != torch.int32 or positions.numel() != T):
+        raise KernelError("head_conv_norm_write: rot_freq is float32 [pairs, 2] inside a head, positions int32 [T]")
+    if D > 256 or E > 256:
+        raise KernelError("head_conv_norm_write: heads are at most 256 wide")
+    if k_pages is not None and (k_pages.dtype != proj.dtype or tuple(k_pages.shape[1:]) != (G, page_tokens, D)
+                                or v_pages is None or tuple(v_pages.shape[1:]) != (G, page_tokens, E)):
+        raise KernelError("head_conv_norm_write: pages are [page, G, page_tokens, D] and [page, G, page_tokens, E]")
+    for x in (request_of_row, q_start, q_len, state_slots):
+        if x.dtype != torch.int32:
+            raise KernelError("head_conv_norm_write: the step's arrays are int32")
+    q = torch.empty((T, H * D), dtype=torch.float32, device=proj.device)
+    ld = proj.stride(0) if T > 1 else max(proj.stride(0), C)
+    fn = _fn("masked_attention", "pbe_head_conv_norm_write",
+             [c_void_p, c_int] + [c_void_p] * 8 + [c_int] * 7 + [c_float, c_void_p, c_void_p, c_int, c_int, c_int]
+             + [c_void_p] * 4 + [c_int, c_void_p])
+    _check(fn(_ptr(proj), ld, _ptr(conv_t), _ptr(conv_state), _ptr(q_gain), _ptr(k_gain),
+              _ptr(slots if k_pages is not None else None), _ptr(q), _ptr(k_pages), _ptr(v_pages), T, int(num_requests),
+              H, G, D, E, int(page_tokens), float(eps), _ptr(positions), _ptr(rot_freq),
+              2 * rot_freq.shape[0] if rot_freq is not None else 0, taps, 1 if update_state else 0,
+              _ptr(request_of_row), _ptr(q_start), _ptr(q_len), _ptr(state_slots), _dtype_code(proj), _stream()),
+           "head_conv_norm_write")
+    if update_state and not single_tokens and taps > 1:
+        conv_state_advance(proj[:, :C], conv_state, q_start, q_len, state_slots, num_requests, skip=1)
+    return q
+
+
+def turn_frequencies(pairs: int, base: float, device, scaling: Optional[dict] = None) -> torch.Tensor:
     """base^(-i / pairs) for i = 0 .. pairs - 1 in turns a position (divided by 2 pi), float32 [pairs, 2]:
-    the rounded number and what the rounding left."""
+    the rounded number and what the rounding left.  ``scaling`` (factor, low, high, original): a pair that
+    turns more than ``high`` times within ``original`` positions keeps its frequency, one that turns less
+    than ``low`` times has it divided by ``factor``, and in between the two are blended linearly in the
+    number of turns."""
     i = torch.arange(pairs, dtype=torch.float64)
     f = torch.pow(torch.tensor(float(base), dtype=torch.float64), -i / pairs) / (2.0 * math.pi)
+    if scaling:
+        factor, low, high = (float(scaling[k]) for k in ("factor", "low", "high"))
+        turns = f * float(scaling["original"])
+        # low == high: a pair on the edge itself keeps the blend's upper end
+        kept = ((turns - low) / (high - low)).clamp(0.0, 1.0) if high > low else (turns >= low).double()
+        f = kept * f + (1.0 - kept) * f / factor
     hi = f.to(torch.float32)
     return torch.stack([hi, (f - hi.double()).to(torch.float32)], dim=1).contiguous().to(device)
 
@@ -1649,15 +1757,17 @@ GROUP_RANKS = {"max": 1, "top2_sum": 2}
 
 
 def route(logits: torch.Tensor, top: int, groups: int, keep: int, scale: float, score: str = "softmax",
-          correction: Optional[torch.Tensor] = None, group_rank: str = "max"):
-    """(chosen int32 [T, top], weights float32 [T, top]) from float32 router logits [T, E]: scores
+          correction: Optional[torch.Tensor] = None, group_rank: str = "max", normalize: bool = True):
+    """(chosen int32 [T, top], weights float32 [T, top]) from float32 router logits [T, E] (columns of a wider
+    matrix may follow): scores
     by ``score`` ("softmax" over the experts or "sigmoid" of each logit); the choice is made on the
     scores plus ``correction`` (float32 [E], optional): experts outside the ``keep`` best of
     ``groups`` neighbouring groups barred (a group ranks by ``group_rank``: its "max" or its
     "top2_sum"), the top ones chosen; weights = score (uncorrected) / (sum of the chosen + 1e-20) *
-    scale."""
+    scale, or score * scale when not ``normalize``."""
     _need_cuda(logits, correction)
-    _need_contiguous(logits, correction)
+    _need_contiguous(correction)
+    _column_slice(logits, "route")
     if score not in ROUTER_SCORES or group_rank not in GROUP_RANKS:
         raise KernelError(f"route: scores are one of {sorted(ROUTER_SCORES)}, group ranks one of {sorted(GROUP_RANKS)}")
     if correction is not None and (correction.dtype != torch.float32 or correction.numel() != logits.shape[1]):
@@ -1669,27 +1779,40 @@ def route(logits: torch.Tensor, top: int, groups: int, keep: int, scale: float, 
         raise KernelError("route: at most 512 experts, 32 chosen and 64 groups")
     chosen = torch.empty((T, top), dtype=torch.int32, device=logits.device)
     weights = torch.empty((T, top), dtype=torch.float32, device=logits.device)
-    fn = _fn("routed_experts", "pbe_route", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
-                                            c_int, c_void_p, c_int, c_void_p])
-    _check(fn(_ptr(logits), _ptr(chosen), _ptr(weights), T, E, int(top), int(groups), int(keep), float(scale),
-              ROUTER_SCORES[score], _ptr(correction), GROUP_RANKS[group_rank], _stream()), "route")
+    fn = _fn("routed_experts", "pbe_route", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
+                                            c_int, c_void_p, c_int, c_int, c_void_p])
+    _check(fn(_ptr(logits), logits.stride(0) if T > 1 else max(logits.stride(0), E), _ptr(chosen), _ptr(weights), T, E, int(top), int(groups), int(keep), float(scale),
+              ROUTER_SCORES[score], _ptr(correction), GROUP_RANKS[group_rank], 1 if normalize else 0, _stream()), "route")
     return chosen, weights
+
+
+def _row_gate(gate: Optional[torch.Tensor], T: int) -> int:
+    """Row stride of a column [T, 1] of float32 numbers (0: there is none)."""
+    if gate is None:
+        return 0
+    _need_cuda(gate)
+    if gate.dtype != torch.float32 or tuple(gate.shape) != (T, 1):
+        raise KernelError("the addend's gate is a float32 column [T, 1]")
+    return gate.stride(0) if T > 1 else 1
 
 
 def expert_rows(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor,
                 chosen: torch.Tensor, weights: torch.Tensor, activation: str = "silu", limit: float = 0.0,
-                alpha: float = 1.0, addend: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """out[t] = (addend[t], optional) + sum_k weights[t, k] * W_down[e] act(W_gate[e] x_t, W_up[e] x_t), e = chosen[t, k]:
+                alpha: float = 1.0, addend: Optional[torch.Tensor] = None, addend_gate: Optional[torch.Tensor] = None,
+                weight_on: str = "output") -> torch.Tensor:
+    """out[t] = (addend[t], optional, times sigmoid(addend_gate[t])) + sum_k weights[t, k] * W_down[e] act(W_gate[e] x_t, W_up[e] x_t), e = chosen[t, k]:
     a block per (row, chosen expert) streams that expert's matrices; for few rows.  ``w_gate_up``
     [E, 2F, W]: an expert's gate rows followed by its up rows; ``w_down`` [E, W, F].  ``activation``:
-    one of ``GLU_ACTIVATIONS`` (see ``gated_activation``)."""
+    one of ``GLU_ACTIVATIONS`` (see ``gated_activation``), or of ``UNGATED_EXPERTS``: W_down relu(W_up x)^2,
+    ``w_gate_up`` is then [E, F, W].  ``weight_on`` "input": the expert reads weight * x_t instead."""
     _need_cuda(x, w_gate_up, w_down, chosen, weights)
     _need_contiguous(x, w_gate_up, w_down, chosen, weights)
     T, W = x.shape
     E, F2, _ = w_gate_up.shape
-    F = F2 // 2
+    ungated = activation in UNGATED_EXPERTS
+    F = F2 if ungated else F2 // 2
     top = chosen.shape[1]
-    if F2 % 2 or tuple(w_down.shape) != (E, W, F) or w_gate_up.shape[2] != W:
+    if (F2 % 2 and not ungated) or tuple(w_down.shape) != (E, W, F) or w_gate_up.shape[2] != W:
         raise KernelError("expert_rows: gate/up is [E, 2F, W], down is [E, W, F]")
     if not (x.dtype == w_gate_up.dtype == w_down.dtype):
         raise KernelError("expert_rows: rows and expert matrices share a dtype")
@@ -1702,12 +1825,17 @@ def expert_rows(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor,
                                or not addend.is_contiguous()):
         raise KernelError("expert_rows: the addend has the rows' shape and dtype")
     fn = _fn("routed_experts", "pbe_expert_rows", [c_void_p] * 3 + [c_ll] + [c_void_p] * 6 + [c_int] * 6 +
-             [c_float, c_float, c_void_p, c_void_p])
+             [c_float, c_float, c_void_p, c_void_p, c_int, c_int, c_void_p])
     global _launches
-    up = c_void_p(w_gate_up.data_ptr() + F * W * w_gate_up.element_size())
-    _check(fn(_ptr(x), _ptr(w_gate_up), up, 2 * F * W, _ptr(w_down), _ptr(chosen), _ptr(weights), _ptr(hidden),
-              _ptr(part), _ptr(out), _dtype_code(x), T, W, F, top, GLU_ACTIVATIONS[activation], float(limit),
-              float(alpha), _ptr(addend), _stream()), "expert_rows")
+    up = c_void_p(w_gate_up.data_ptr() + (F2 - F) * W * w_gate_up.element_size())
+    act = UNGATED_EXPERTS[activation] if ungated else GLU_ACTIVATIONS[activation]
+    if activation not in ("silu", "capped_swish") and not ungated:
+        raise KernelError(f"expert_rows: no expert activation {activation!r}")
+    gate_ld = _row_gate(addend_gate, T)
+    _check(fn(_ptr(x), _ptr(w_gate_up), up, F2 * W, _ptr(w_down), _ptr(chosen), _ptr(weights), _ptr(hidden),
+              _ptr(part), _ptr(out), _dtype_code(x), T, W, F, top, act, float(limit),
+              float(alpha), _ptr(addend), _ptr(addend_gate), gate_ld, 1 if weight_on == "input" else 0, _stream()),
+           "expert_rows")
     _launches += 2
     return out
 
@@ -1726,8 +1854,9 @@ def expert_places(chosen: torch.Tensor, num_experts: int):
 
 
 def expert_gather(x: torch.Tensor, chosen: torch.Tensor, place: torch.Tensor, start: torch.Tensor,
-                  total_rows: Optional[int] = None) -> torch.Tensor:
-    """The rows of x once per chosen expert, sorted by expert: row start[e] + place[pair] = x[t].
+                  total_rows: Optional[int] = None, weights: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """The rows of x once per chosen expert, sorted by expert: row start[e] + place[pair] = x[t] (times
+    ``weights[t, k]``, float32, when given).
     ``total_rows``: rows of the result when the experts' runs are padded (rows between the runs are
     left as they are)."""
     _need_cuda(x, chosen, place, start)
@@ -1735,16 +1864,18 @@ def expert_gather(x: torch.Tensor, chosen: torch.Tensor, place: torch.Tensor, st
     T, W = x.shape
     top = chosen.shape[1]
     out = torch.empty((total_rows or T * top, W), dtype=x.dtype, device=x.device)
-    fn = _fn("routed_experts", "pbe_expert_gather", [c_void_p] * 5 + [c_int] * 4 + [c_void_p])
-    _check(fn(_ptr(x), _ptr(chosen), _ptr(place), _ptr(start), _ptr(out), _dtype_code(x), T, top, W, _stream()),
+    fn = _fn("routed_experts", "pbe_expert_gather", [c_void_p] * 6 + [c_int] * 4 + [c_void_p])
+    _check(fn(_ptr(x), _ptr(chosen), _ptr(place), _ptr(start), _ptr(weights), _ptr(out), _dtype_code(x), T, top, W, _stream()),
            "expert_gather")
     return out
 
 
 def expert_scatter(y: torch.Tensor, chosen: torch.Tensor, place: torch.Tensor, start: torch.Tensor,
-                   weights: torch.Tensor, T: int, addend: Optional[torch.Tensor] = None) -> torch.Tensor:
+                   weights: Optional[torch.Tensor], T: int, addend: Optional[torch.Tensor] = None,
+                   addend_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """out[t] = sum_k weights[t, k] * y[start[e] + place[(t, k)]], e = chosen[t, k], in k order, plus
-    ``addend`` [T, W] (optional, y's dtype)."""
+    ``addend`` [T, W] (optional, y's dtype), times sigmoid(``addend_gate``) (a float32 column [T, 1]) when
+    given.  ``weights`` None: all one."""
     _need_cuda(y, chosen, place, start, weights, addend)
     _need_contiguous(y, chosen, place, start, weights, addend)
     if addend is not None and (tuple(addend.shape) != (T, y.shape[1]) or addend.dtype != y.dtype):
@@ -1752,9 +1883,9 @@ def expert_scatter(y: torch.Tensor, chosen: torch.Tensor, place: torch.Tensor, s
     W = y.shape[1]
     top = chosen.shape[1]
     out = torch.empty((T, W), dtype=y.dtype, device=y.device)
-    fn = _fn("routed_experts", "pbe_expert_scatter", [c_void_p] * 6 + [c_int] * 4 + [c_void_p, c_void_p])
+    fn = _fn("routed_experts", "pbe_expert_scatter", [c_void_p] * 6 + [c_int] * 4 + [c_void_p, c_void_p, c_int, c_void_p])
     _check(fn(_ptr(y), _ptr(chosen), _ptr(place), _ptr(start), _ptr(weights), _ptr(out), _dtype_code(y), T, top, W,
-              _ptr(addend), _stream()), "expert_scatter")
+              _ptr(addend), _ptr(addend_gate), _row_gate(addend_gate, T), _stream()), "expert_scatter")
     return out
 
 
@@ -1763,20 +1894,23 @@ GROUP_TILE_ROWS = 64     # rows of a tile of the grouped product (runs of rows a
 
 
 def _grouped(a, lda, a_group, w, w_group, wk, wn, out, ldo, out_group, T, K, N, groups, tiles, num_tiles,
-             gate=None, rot=0, rot_dims=0, inv_freq=None, positions=None, rot_scale=1.0, gate_each=False):
+             gate=None, rot=0, rot_dims=0, inv_freq=None, positions=None, rot_scale=1.0, gate_each=False,
+             activation=None):
     _need_cuda(a, w, out, tiles, gate, inv_freq, positions)
     if w.dtype != torch.bfloat16 or (gate is not None and (gate.dtype != torch.bfloat16 or gate.stride(1) != 1)):
         raise KernelError("grouped product: weights (and the gate) are bfloat16")
     fn = _fn("grouped_gemm", "pbe_grouped_gemm",
              [c_void_p, c_int, c_int, c_ll, c_void_p, c_ll, c_int, c_int, c_void_p, c_int, c_int, c_ll, c_int, c_int, c_int,
-              c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_int, c_void_p])
+              c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_int, c_int, c_void_p])
+    if activation not in (None, "relu2"):
+        raise KernelError(f"grouped product: no epilogue {activation!r}")
     ldg = 0
     if gate is not None:
         ldg = gate.stride(0) if T > 1 else max(gate.stride(0), groups * (N if gate_each else 1))
     _check(fn(_ptr(a), _dtype_code(a), int(lda), int(a_group), _ptr(w), int(w_group), int(wk), int(wn), _ptr(out),
               _dtype_code(out), int(ldo), int(out_group), int(T), int(K), int(N), int(groups), _ptr(tiles),
               int(num_tiles), _ptr(gate), int(ldg), int(rot), int(rot_dims), _ptr(inv_freq), _ptr(positions),
-              float(rot_scale), 1 if gate_each else 0, _stream()), "grouped_gemm")
+              float(rot_scale), 1 if gate_each else 0, 1 if activation == "relu2" else 0, _stream()), "grouped_gemm")
     return out
 
 
@@ -1804,8 +1938,9 @@ def run_tiles(counts: torch.Tensor, max_tiles: int):
     return start, tiles
 
 
-def grouped_runs(a: torch.Tensor, w: torch.Tensor, tiles: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
-    """out[row] = W[g] a[row] for the rows of every tile (group g): ``a`` [rows, K] sorted by group,
+def grouped_runs(a: torch.Tensor, w: torch.Tensor, tiles: torch.Tensor, out_dtype: torch.dtype,
+                 activation: Optional[str] = None) -> torch.Tensor:
+    """out[row] = W[g] a[row] (with ``activation`` "relu2" its relu squared) for the rows of every tile (group g): ``a`` [rows, K] sorted by group,
     ``w`` bfloat16 [G, N, K], ``tiles`` from ``run_tiles``."""
     _need_contiguous(a, w, tiles)
     rows, K = a.shape
@@ -1813,7 +1948,7 @@ def grouped_runs(a: torch.Tensor, w: torch.Tensor, tiles: torch.Tensor, out_dtyp
     if w.shape[2] != K:
         raise KernelError("grouped_runs: the weights are [G, N, K]")
     out = torch.empty((rows, N), dtype=out_dtype, device=a.device)
-    return _grouped(a, K, 0, w, N * K, 1, K, out, N, 0, rows, K, N, G, tiles, tiles.shape[0])
+    return _grouped(a, K, 0, w, N * K, 1, K, out, N, 0, rows, K, N, G, tiles, tiles.shape[0], activation=activation)
 
 
 # ------------------------------------------------------------------ norms with one learned number, mix over depth
@@ -2106,4 +2241,98 @@ def delta_scan(qk: torch.Tensor, kq: torch.Tensor, v: torch.Tensor, beta: torch.
     _check(fn(_ptr(qk), _ptr(kq), _ptr(v), _ptr(beta), _ptr(decay), 1 if per_channel else 0, _ptr(out), _ptr(state),
               _ptr(q_start), _ptr(q_len), _ptr(slots), int(num_requests), G, H, D, E, 1 if update_state else 0,
               _stream()), "delta_scan")
+    return out
+
+
+# ------------------------------------------------------------------ time mixing (a decay per channel, a bonus)
+def token_shift(h: torch.Tensor, mu: torch.Tensor, state: torch.Tensor, request_of_row: torch.Tensor,
+                q_start: torch.Tensor, q_len: torch.Tensor, slots: torch.Tensor, num_requests: int,
+                update_state: bool = True) -> torch.Tensor:
+    """out[s, t] = h[t] + (h[t - 1] - h[t]) * mu[s] for ``mu`` float32 [S, W]; the row before a request's first
+    row of the step is its row of ``state`` (float32 [slots, W]), which its last row then replaces
+    (``update_state``).  Returns [S, T, W] in h's dtype; padding rows become zeros."""
+    _need_cuda(h, mu, state, request_of_row, q_start, q_len, slots)
+    _need_contiguous(h, mu, state)
+    T, W = h.shape
+    if mu.dtype != torch.float32 or mu.dim() != 2 or mu.shape[1] != W or not 1 <= mu.shape[0] <= 8:
+        raise KernelError("token_shift: mu is float32 [S, W] with one to eight rows")
+    if state.dtype != torch.float32 or tuple(state.shape[1:]) != (W,):
+        raise KernelError("token_shift: the state is float32 [slots, W]")
+    for x in (request_of_row, q_start, q_len, slots):
+        if x.dtype != torch.int32:
+            raise KernelError("token_shift: the step's arrays are int32")
+    out = torch.empty((mu.shape[0], T, W), dtype=h.dtype, device=h.device)
+    fn = _fn("time_mixing", "pbe_token_shift", [c_void_p, c_int] + [c_void_p] * 7 + [c_int] * 5 + [c_void_p])
+    _check(fn(_ptr(h), _dtype_code(h), _ptr(mu), _ptr(state), _ptr(out), _ptr(request_of_row), _ptr(q_start), _ptr(q_len),
+              _ptr(slots), T, int(num_requests), W, mu.shape[0], 1 if update_state else 0, _stream()), "token_shift")
+    return out
+
+
+def low_rank_decay(x: torch.Tensor, w2_t: torch.Tensor, w0: torch.Tensor) -> torch.Tensor:
+    """exp(-exp(w0 + tanh(x) w2_t)), float32 [T, C]: ``x`` float32 [T, rank], ``w2_t`` [rank, C] in float32 or
+    bfloat16, ``w0`` float32 [C]; float32 arithmetic."""
+    _need_cuda(x, w2_t, w0)
+    _need_contiguous(w2_t, w0)
+    _column_slice(x, "low_rank_decay")
+    T, rank = x.shape
+    C = w2_t.shape[1]
+    if x.dtype != torch.float32 or w2_t.shape[0] != rank or w0.dtype != torch.float32 or w0.numel() != C:
+        raise KernelError("low_rank_decay: x is float32 [T, rank], w2_t [rank, C], w0 float32 [C]")
+    decay = torch.empty((T, C), dtype=torch.float32, device=x.device)
+    fn = _fn("time_mixing", "pbe_low_rank_decay", [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
+                                                   c_int, c_void_p])
+    _check(fn(_ptr(x), x.stride(0) if T > 1 else max(x.stride(0), rank), _ptr(w2_t), _dtype_code(w2_t), _ptr(w0), _ptr(decay),
+              T, C, rank, _stream()), "low_rank_decay")
+    return decay
+
+
+WKV_CHUNK_MAX_DIM = 256       # wider key heads always run token by token
+
+
+def wkv(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, bonus: torch.Tensor,
+        state: torch.Tensor, q_start: torch.Tensor, q_len: torch.Tensor, slots: torch.Tensor, num_requests: int,
+        heads: int, update_state: bool = True, zero_out: bool = False, chunked: bool = False) -> torch.Tensor:
+    """o_t = (S + diag(bonus) k_t v_t^T)^T r_t, S <- diag(decay_t) S + k_t v_t^T per head, request by request over
+    the rows each brings: ``r``, ``k`` [T, H * D] and ``v`` [T, H * E] column slices in one dtype, ``decay`` float32
+    [T, H * D] (numbers in [0, 1]), ``bonus`` float32 [H * D], ``state`` float32 [slots, H, E, D] (S transposed: a
+    value column's key channels side by side), read at ``slots[r]`` and left updated.  ``chunked``: sixteen
+    tokens at a time (prompt portions: two launches), else one by one.  Returns o, float32 [T, H * E]."""
+    _need_cuda(r, k, v, decay, bonus, state, q_start, q_len, slots)
+    _need_contiguous(decay, bonus, state)
+    for x in (r, k, v):
+        _column_slice(x, "wkv")
+    T, H = r.shape[0], heads
+    D, E = r.shape[1] // H, v.shape[1] // H
+    if k.shape != r.shape or r.shape[1] != H * D or tuple(v.shape) != (T, H * E) or r.dtype != k.dtype or \
+            r.dtype != v.dtype or tuple(decay.shape) != (T, H * D) or bonus.numel() != H * D or \
+            tuple(state.shape[1:]) != (H, E, D):
+        raise KernelError("wkv: shapes or dtypes do not agree")
+    for x in (decay, bonus, state):
+        if x.dtype != torch.float32:
+            raise KernelError("wkv: decays, bonus and state are float32")
+    if D > 512:
+        raise KernelError(f"wkv: key width {D} per head is beyond 512")
+    for x in (q_start, q_len, slots):
+        if x.dtype != torch.int32 or x.numel() < num_requests:
+            raise KernelError("wkv: request arrays are int32 [R]")
+
+    def ld(x):
+        return x.stride(0) if T > 1 else max(x.stride(0), x.shape[1])
+    out = (torch.zeros if zero_out else torch.empty)((T, H * E), dtype=torch.float32, device=v.device)
+    heads_of = [_ptr(r), _ptr(k), _ptr(v), ld(r), ld(k), ld(v), _dtype_code(r), _ptr(decay), _ptr(bonus), _ptr(out),
+                _ptr(state)]
+    types = [c_void_p] * 3 + [c_int] * 4 + [c_void_p] * 4
+    if chunked and D <= WKV_CHUNK_MAX_DIM:
+        size = _fn("time_mixing", "pbe_wkv_record_floats", [c_int])(D)
+        ct = _fn("time_mixing", "pbe_wkv_chunk_tokens", [])()
+        records = torch.empty((T // ct + int(num_requests), H, size), dtype=torch.float32, device=v.device)
+        fn = _fn("time_mixing", "pbe_wkv_chunks", types + [c_void_p] * 4 + [c_int] * 6 + [c_void_p])
+        global _launches
+        _check(fn(*heads_of, _ptr(records), _ptr(q_start), _ptr(q_len), _ptr(slots), T, int(num_requests), H, D, E,
+                  1 if update_state else 0, _stream()), "wkv_chunks")
+        _launches += 1
+        return out
+    fn = _fn("time_mixing", "pbe_wkv_steps", types + [c_void_p] * 3 + [c_int] * 5 + [c_void_p])
+    _check(fn(*heads_of, _ptr(q_start), _ptr(q_len), _ptr(slots), int(num_requests), H, D, E, 1 if update_state else 0,
+              _stream()), "wkv_steps")
     return out

@@ -114,8 +114,7 @@ class DecoderModel:
         for step in self.spec.run_order:
             mixer = self.blocks[step.block].mixer
             lc = storage.layer(step.cache_layer)
-            for gsize, tile_rows, window in mixer.work_keys():
-                key = (lc.group, gsize, tile_rows, window)
+            for key in mixer.paged_work(lc):
                 if key not in keys:
                     keys.append(key)
         return keys

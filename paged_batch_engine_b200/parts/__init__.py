@@ -1,11 +1,11 @@
 from .base import (Block, CacheTensor, CompositeNeed, FeedForward, KVNeed, Mixer, Norm, PagedNeed, Part, PositionEncoding, StateNeed,
                    build_block, build_part, register_part)
-from .norm import DeltaSum, LayerNorm, PendingUpdate, RMSNorm, ScalarRMSNorm
+from .norm import DeltaSum, LayerNorm, NormedDelta, PendingUpdate, RMSNorm, ScalarRMSNorm
 from .rope import NoPositionEncoding, RotaryEncoding
 from .attention import GQAttention
 from .mlp import ActivationMLP, SwiGLU
 from .routed_experts import RoutedExperts
-from .block import DepthStack, OutputNormBlock, ParallelBlock, PostNormBlock, PreNormBlock
+from .block import DepthStack, OutputNormBlock, ParallelBlock, PostNormBlock, PreNormBlock, SandwichBlock
 from .gated_recurrence import GatedLinearRecurrence
 from .delta_rule import GatedDeltaRule
 from .linear_attention import DecayLinearAttention
@@ -14,6 +14,7 @@ from .parallel import ParallelMixer
 from .state_space import SelectiveStateSpace
 from .latent_attention import LatentAttention
 from .masked_attention import MaskedAttention
+from .time_mixing import TimeMixing
 from .streams import StreamBlock, StreamConnection
 
 __all__ = ["Block", "CacheTensor", "CompositeNeed", "FeedForward", "KVNeed", "Mixer", "Norm", "PagedNeed", "Part", "PositionEncoding",
@@ -23,4 +24,4 @@ __all__ = ["Block", "CacheTensor", "CompositeNeed", "FeedForward", "KVNeed", "Mi
            "PooledWindowAttention", "ParallelMixer", "StreamBlock", "StreamConnection", "DeltaSum", "ActivationMLP",
            "RoutedExperts", "ParallelBlock", "SelectiveStateSpace", "LatentAttention", "MaskedAttention",
            "ScalarRMSNorm", "DepthStack", "PostNormBlock", "GatedLinearRecurrence",
-           "OutputNormBlock", "GatedDeltaRule"]
+           "OutputNormBlock", "GatedDeltaRule", "NormedDelta", "SandwichBlock", "TimeMixing"]

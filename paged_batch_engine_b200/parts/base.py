@@ -136,6 +136,11 @@ class Mixer(Part):
         tile rows, window) triples."""
         return []
 
+    def paged_work(self, cache):
+        """The work lists with the layer group each reads, (group, heads per kv head, tile rows, window);
+        ``cache``: the mixer's ``LayerCache``.  A mixer whose pages are a part of a composite need says which."""
+        return [(cache.group,) + tuple(k) for k in self.work_keys()]
+
     def forward(self, x, ctx, cache):
         raise NotImplementedError
 

@@ -6,7 +6,7 @@ import torch
 from ..config.specs import BlockSpec
 from .base import Block, build_part, register_part
 from ..weights.loader import ParamSpec
-from .norm import DeltaSum
+from .norm import DeltaSum, NormedDelta
 
 
 class PreNormBlock(Block):
@@ -282,6 +282,48 @@ class OutputNormBlock(Block):
         return st, None
 
 
+class SandwichBlock(PreNormBlock):
+    """A norm before and after each sublayer: x <- x + n1b(mixer(n1(x))), then (with a feed-forward)
+    x <- x + n2b(feed_forward(n2(x))).  The norm behind a sublayer, the sum and the norm ahead of the next
+    one are one launch: the sublayer's output travels to it as a ``NormedDelta``, from layer to layer too.
+    ``names`` gives the later norms' tensors as "norm_mixer_out" and "norm_feed_forward_out"."""
+
+    def __init__(self, spec: BlockSpec, dtype, device):
+        self.spec = spec
+        self.prefix = spec.prefix
+        n = spec.names
+        self.p_mixer = self.prefix + n.get("mixer", "mixer.")
+        self.p_ffn = self.prefix + n.get("feed_forward", "feed_forward.")
+        self.p_norm1 = self.prefix + n.get("norm_mixer", "norm_mixer.")
+        self.p_norm1b = self.prefix + n.get("norm_mixer_out", "norm_mixer_out.")
+        self.p_norm2 = self.prefix + n.get("norm_feed_forward", "norm_feed_forward.")
+        self.p_norm2b = self.prefix + n.get("norm_feed_forward_out", "norm_feed_forward_out.")
+        self.norm1 = build_part("norm", spec.norm_mixer, dtype, device)
+        self.norm1b = build_part("norm", spec.args.get("norm_mixer_out", spec.norm_mixer), dtype, device)
+        self.mixer = build_part("mixer", spec.mixer, dtype, device)
+        self.norm2 = self.norm2b = self.ffn = None
+        if spec.feed_forward is not None:
+            self.norm2 = build_part("norm", spec.norm_feed_forward, dtype, device)
+            self.norm2b = build_part("norm", spec.args.get("norm_feed_forward_out", spec.norm_feed_forward), dtype, device)
+            self.ffn = build_part("feed_forward", spec.feed_forward, dtype, device)
+        for norm in (self.norm1, self.norm1b, self.norm2, self.norm2b):
+            if norm is not None and not (hasattr(norm, "norm_add") and norm.on_output):
+                raise TypeError("a sandwich block needs norms that chain behind a norm (RMSNorm with on_output)")
+
+    def parts(self):
+        out = [(self.norm1, self.p_norm1), (self.mixer, self.p_mixer), (self.norm1b, self.p_norm1b)]
+        if self.ffn is not None:
+            out += [(self.norm2, self.p_norm2), (self.ffn, self.p_ffn), (self.norm2b, self.p_norm2b)]
+        return out
+
+    def forward(self, residual, delta, ctx, cache):
+        y = NormedDelta(self.mixer.forward(self.norm1.add_norm(residual, delta), ctx, cache), self.norm1b)
+        if self.ffn is not None:
+            y = NormedDelta(self.ffn.forward(self.norm2.add_norm(residual, y), ctx), self.norm2b)
+        return residual, y
+
+
+register_part("block", "sandwich", lambda spec, dtype, device: SandwichBlock(spec, dtype, device), replace=True)
 register_part("block", "outnorm", lambda spec, dtype, device: OutputNormBlock(spec, dtype, device), replace=True)
 register_part("block", "postnorm", lambda spec, dtype, device: PostNormBlock(spec, dtype, device), replace=True)
 register_part("block", "prenorm", lambda spec, dtype, device: PreNormBlock(spec, dtype, device),

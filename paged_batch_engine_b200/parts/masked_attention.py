@@ -9,7 +9,7 @@ import torch
 
 from ..csrc import ops
 from ..weights.loader import ParamSpec
-from .base import CacheTensor, Mixer, PagedNeed, register_part
+from .base import CacheTensor, CompositeNeed, Mixer, PagedNeed, StateNeed, register_part
 
 
 def log_bucket(distance: int, rows: int, far: float) -> int:
@@ -43,7 +43,10 @@ class MaskedAttention(Mixer):
     ``softcap`` c: the scaled score becomes c tanh(score / c) before the bias is added.
     ``rotary`` dict(dims=n, base=b): after the norm the first n dimensions of every query and key turn by
     the token's position, dimension i with i + n/2 by position * b^(-2i/n) (halves paired); keys are
-    cached so.  ``rotate_values``: the value of position j turns by j over all ``value_dim`` dimensions in
+    cached so.  An entry ``scaling`` (factor, low, high, original) stretches slow pairs (see
+    ``ops.turn_frequencies``).  ``conv_taps`` n: a causal convolution per channel of q, k and v (n taps, no
+    bias, the last one on the current token) between the projection and the norm, tensors ``.conv`` [channels,
+    n]; the last n - 1 projected rows are kept per request in float32.  ``rotate_values``: the value of position j turns by j over all ``value_dim`` dimensions in
     the same way (base ``rotary["base"]``) and is cached so; each head's output at position i turns back
     by i, ahead of the gate.
     ``out_gate``: the concatenated heads are multiplied by sigmoid(W_g x) element by element.
@@ -57,7 +60,7 @@ class MaskedAttention(Mixer):
     [hidden, H*E], q.norm / k.norm [D], rel [B, H], sink [H], g [H*E, hidden], and ``.b`` beside q, k, v, o
     (``tensor_names`` renames them)."""
     TENSOR_NAMES = dict(q="q", k="k", v="v", o="o", q_norm="q.norm", k_norm="k.norm", rel="rel", g="g",
-                        temp="temp", sink="sink", bias_suffix=".b")
+                        temp="temp", sink="sink", bias_suffix=".b", conv_suffix=".conv")
     decode_capturable = True      # stepped from the step's device arrays alone
 
     def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, key_dim: int, value_dim: int,
@@ -65,7 +68,8 @@ class MaskedAttention(Mixer):
                  mask_size: Optional[int] = None, qk_norm: bool = True, distance_bias: Optional[dict] = None,
                  unit_sink: bool = False, out_gate: bool = False, proj_bias=False,
                  head_temperature: bool = False, sink: bool = False, softcap: Optional[float] = None,
-                 rotary: Optional[dict] = None, rotate_values: bool = False, tensor_names: Optional[dict] = None):
+                 rotary: Optional[dict] = None, rotate_values: bool = False, conv_taps: Optional[int] = None,
+                 tensor_names: Optional[dict] = None):
         unknown = set(tensor_names or {}) - set(self.TENSOR_NAMES)
         if unknown:
             raise ValueError(f"tensor_names knows {sorted(self.TENSOR_NAMES)}; got {sorted(unknown)}")
@@ -105,6 +109,14 @@ class MaskedAttention(Mixer):
             raise ValueError("rotary dims are even, at least 2 and at most the key width")
         if self.rotate_values and (not rotary or value_dim % 2):
             raise ValueError("rotated values take the base of the rotation and an even width")
+        self.rot_scaling = dict(rotary["scaling"]) if rotary and rotary.get("scaling") else None
+        self.conv_taps = int(conv_taps) if conv_taps is not None else 0
+        if self.conv_taps:
+            if not 1 <= self.conv_taps <= 16:
+                raise ValueError("the convolutions have 1 to 16 taps")
+            if self.proj_bias or self.head_temperature or self.rotate_values:
+                raise ValueError("convolutions go with neither projection biases, temperatures nor rotated values")
+        self.conv_t = None
         self.dtype, self.device = dtype, device
         self.rot_freq = self.value_freq = self.sink_scores = None
         self.tile_rows = ops.masked_tile_rows(dtype, key_dim, value_dim)
@@ -114,14 +126,22 @@ class MaskedAttention(Mixer):
     # ---- what it keeps
     def cache_need(self):
         G = self.num_kv_heads
-        return PagedNeed((CacheTensor("k", G, self.key_dim), CacheTensor("v", G, self.value_dim)),
-                         window=self.mask_size)
+        pages = PagedNeed((CacheTensor("k", G, self.key_dim), CacheTensor("v", G, self.value_dim)),
+                          window=self.mask_size)
+        if self.conv_taps < 2:
+            return pages
+        channels = self._columns()[3]
+        return CompositeNeed.of(pages=pages, conv=StateNeed((self.conv_taps - 1, channels), torch.float32))
 
     def work_keys(self):
         return [(self.num_heads // self.num_kv_heads, self.tile_rows, self.mask_size)]
 
+    def paged_work(self, cache):
+        return super().paged_work(cache.sub["pages"] if self.conv_taps > 1 else cache)
+
     def kernel_libraries(self, dtype):
-        return ops.masked_libraries(dtype, self.key_dim, self.value_dim) + ops.gemm_libraries(dtype)
+        conv = [("short_conv", None)] if self.conv_taps > 1 else []
+        return ops.masked_libraries(dtype, self.key_dim, self.value_dim) + conv + ops.gemm_libraries(dtype)
 
     # ---- tensors
     def _columns(self):
@@ -140,6 +160,9 @@ class MaskedAttention(Mixer):
                       ParamSpec(prefix + n["v"] + b, (G * E,))]
             if self.proj_bias is True:
                 specs.append(ParamSpec(prefix + n["o"] + b, (w,)))
+        if self.conv_taps:
+            specs += [ParamSpec(prefix + n[x] + n["conv_suffix"], (rows, self.conv_taps))
+                      for x, rows in (("q", H * D), ("k", G * D), ("v", G * E))]
         if self.qk_norm is True:
             specs += [ParamSpec(prefix + n["q_norm"], (D,)), ParamSpec(prefix + n["k_norm"], (D,))]
         if self.head_temperature:
@@ -164,6 +187,9 @@ class MaskedAttention(Mixer):
         self.w_in = torch.cat(ws, dim=0).contiguous()
         del ws
         self.w_o = tensors.pop(prefix + n["o"]).contiguous()
+        if self.conv_taps:
+            self.conv_t = torch.cat([tensors.pop(prefix + n[x] + n["conv_suffix"]).to(torch.float32) for x in "qkv"],
+                                    dim=0).t().contiguous()          # [taps, channels of q, k and v]
         if self.proj_bias:
             self.b_in = torch.cat([tensors.pop(prefix + n[x] + b).to(torch.float32) for x in "qkv"]).contiguous()
             if self.proj_bias is True:
@@ -178,7 +204,8 @@ class MaskedAttention(Mixer):
         if self.sink:
             self.sink_scores = tensors.pop(prefix + n["sink"]).to(torch.float32).contiguous()
         if self.rot_dims:
-            self.rot_freq = ops.turn_frequencies(self.rot_dims // 2, self.rot_base, self.w_in.device)
+            self.rot_freq = ops.turn_frequencies(self.rot_dims // 2, self.rot_base, self.w_in.device,
+                                                 self.rot_scaling)
         if self.rotate_values:
             self.value_freq = ops.turn_frequencies(self.value_dim // 2, self.rot_base, self.w_in.device)
         if self.bias_rows:
@@ -196,13 +223,28 @@ class MaskedAttention(Mixer):
         H, G, D, E = self.num_heads, self.num_kv_heads, self.key_dim, self.value_dim
         q_off, k_off, v_off, g_off = self._columns()
         proj = ops.linear(x, self.w_in, None, out_dtype=self.dtype, kind=1)
+        conv_state = None
+        if self.conv_taps > 1:
+            conv_state, cache = cache.sub["conv"].state, cache.sub["pages"]
+        elif self.conv_taps:
+            conv_state = torch.empty((1, 0, q_off + v_off + G * E), dtype=torch.float32, device=x.device)
         group = ctx.group(cache.group)
         writes = cache.writes
-        q = ops.head_norm_write(proj, q_off, k_off, v_off, self.b_in, self.q_gain, self.k_gain,
-                                group.slots if writes else None, cache.k if writes else None,
-                                cache.v if writes else None, H, G, D, E, ctx.page_tokens, self.eps,
-                                q_head_scale=self.q_head_scale, positions=ctx.position_ids if self.rot_dims else None,
-                                rot_freq=self.rot_freq, value_freq=self.value_freq)
+        if self.conv_taps:
+            single = getattr(ctx, "captured", False) or ctx.num_tokens == ctx.num_requests
+            q = ops.head_conv_norm_write(
+                proj, self.conv_t, conv_state, self.q_gain, self.k_gain, group.slots if writes else None,
+                cache.k if writes else None, cache.v if writes else None, H, G, D, E, ctx.page_tokens, self.eps,
+                ctx.request_of_row, ctx.q_start, ctx.q_len, ctx.state_slots, ctx.num_requests,
+                positions=ctx.position_ids if self.rot_dims else None, rot_freq=self.rot_freq, update_state=writes,
+                single_tokens=single)
+        else:
+            q = ops.head_norm_write(proj, q_off, k_off, v_off, self.b_in, self.q_gain, self.k_gain,
+                                    group.slots if writes else None, cache.k if writes else None,
+                                    cache.v if writes else None, H, G, D, E, ctx.page_tokens, self.eps,
+                                    q_head_scale=self.q_head_scale,
+                                    positions=ctx.position_ids if self.rot_dims else None,
+                                    rot_freq=self.rot_freq, value_freq=self.value_freq)
         q, turn = q if self.rotate_values else (q, None)
         meta = ctx.attention_work(cache.group, H // G, self.tile_rows, self.mask_size, H, E)
         gate = proj[:, g_off:] if self.out_gate else None

@@ -18,7 +18,8 @@ class RMSNorm(Norm):
     one launch and the residual stream stays float32.
 
     ``one_plus``: the checkpoint stores the gain around zero, w = 1 + stored (formed once at load,
-    in float32).  ``on_output``: the norm sits on a sublayer's output (``norm_add``)."""
+    in float32).  ``on_output``: the norm sits on a sublayer's output (``norm_add``, or left to the next norm's
+    launch as a ``NormedDelta``)."""
 
     def __init__(self, size: int, eps: float, dtype, device, weight_name: str = "weight", one_plus: bool = False,
                  on_output: bool = False):
@@ -38,7 +39,15 @@ class RMSNorm(Norm):
             self.gain = (self.gain + 1.0).contiguous()
 
     def add_norm(self, residual, delta, rows=None, out_dtype=None):
+        if isinstance(delta, NormedDelta):
+            y, n = delta.y, delta.norm
+            a, b, sa, sb = (y.a, y.b, y.scale, y.scale_b) if isinstance(y, DeltaSum) else (y, None, 1.0, 0.0)
+            if a.dtype != (out_dtype or self.dtype):
+                raise ValueError("the norm after a normed sum writes the sublayers' dtype")
+            return ops.norm_add_norm(residual, a, b, sa, sb, n.gain, n.eps, self.gain, self.eps, rows)
         if isinstance(delta, DeltaSum):
+            if delta.scale_b != delta.scale:
+                raise ValueError("this norm adds branches of one common scale")
             return ops.add2_rmsnorm2(residual, delta.a, delta.b, self.gain, None, self.eps,
                                      out_dtype or self.dtype, rows, delta_scale=delta.scale)[0]
         n = residual.shape[0] if rows is None else rows.numel()
@@ -56,6 +65,8 @@ class RMSNorm(Norm):
         if other.size != self.size or other.eps != self.eps:
             raise ValueError("two norms of one row share its width and eps")
         a, b, scale = (delta.a, delta.b, delta.scale) if isinstance(delta, DeltaSum) else (delta, None, 1.0)
+        if isinstance(delta, NormedDelta) or (b is not None and delta.scale_b != scale):
+            raise ValueError("two norms of one row take a plain delta or branches of one common scale")
         return ops.add2_rmsnorm2(residual, a, b, self.gain, other.gain, self.eps, out_dtype or self.dtype,
                                  delta_scale=scale)
 
@@ -82,7 +93,7 @@ class ScalarRMSNorm(Norm):
 
     def add_norm(self, residual, delta, rows=None, out_dtype=None):
         if isinstance(delta, DeltaSum):
-            if delta.scale != 1.0:
+            if delta.scale != 1.0 or delta.scale_b != 1.0:
                 raise ValueError("a norm with one gain adds unscaled branches")
             a, b = delta.a, delta.b
         else:
@@ -167,12 +178,22 @@ class LayerNorm(Norm):
 
 
 class DeltaSum:
-    """Two branch outputs of one layer that are not yet added to the residual: x' = x + scale *
-    (a + b) (``b`` may be None).  The next norm's launch adds them."""
-    __slots__ = ("a", "b", "scale")
+    """Two branch outputs of one layer that are not yet added to the residual: x' = x + scale * a +
+    scale_b * b (``b`` may be None; ``scale_b`` None: one scale for both).  The next norm's launch adds them."""
+    __slots__ = ("a", "b", "scale", "scale_b")
 
-    def __init__(self, a, b, scale: float = 1.0):
+    def __init__(self, a, b, scale: float = 1.0, scale_b: Optional[float] = None):
         self.a, self.b, self.scale = a, b, float(scale)
+        self.scale_b = self.scale if scale_b is None else float(scale_b)
+
+
+class NormedDelta:
+    """A sublayer's output ``y`` (a tensor or a ``DeltaSum``) whose norm is not yet added to the residual:
+    x' = x + norm(y).  The next norm's launch forms both."""
+    __slots__ = ("y", "norm")
+
+    def __init__(self, y, norm):
+        self.y, self.norm = y, norm
 
 
 class PendingUpdate:

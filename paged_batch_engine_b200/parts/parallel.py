@@ -1,7 +1,7 @@
 """Several mixers side by side on the same input."""
 from __future__ import annotations
 
-from typing import Sequence, Tuple
+from typing import Optional, Sequence, Tuple
 
 import torch
 
@@ -9,6 +9,7 @@ from ..config.specs import PartSpec
 from ..csrc import ops
 from ..weights.loader import ParamSpec
 from .base import CompositeNeed, Mixer, build_part, register_part
+from .norm import DeltaSum
 
 
 class ParallelMixer(Mixer):
@@ -18,12 +19,20 @@ class ParallelMixer(Mixer):
 
     ``branches``: (name, PartSpec) pairs; branch ``name`` has its tensors under ``prefix + name +
     "."`` and its gain at ``prefix + name + "." + gain_name``; each branch keeps a cache of its
-    own kind (the parts of a ``CompositeNeed`` by branch name)."""
+    own kind (the parts of a ``CompositeNeed`` by branch name).
+
+    ``combine`` "sum": y = sum over the (one or two) branches of scale_b * out_b, with the constants
+    ``scales`` and no gain tensors; the sum is left to the launch that reads it (a ``DeltaSum``)."""
 
     def __init__(self, hidden_size: int, branches: Sequence[Tuple[str, PartSpec]], eps: float, dtype, device,
-                 gain_name: str = "out"):
+                 gain_name: str = "out", combine: str = "rms_mean", scales: Optional[Sequence[float]] = None):
         if not 1 <= len(branches) <= 4:
             raise ValueError("one to four branches")
+        if combine not in ("rms_mean", "sum"):
+            raise ValueError(f"unknown combine {combine!r}; known: rms_mean, sum")
+        if combine == "sum" and (len(branches) > 2 or scales is None or len(scales) != len(branches)):
+            raise ValueError("a scaled sum has one or two branches and a scale for each")
+        self.combine, self.scales = combine, [float(x) for x in scales or ()]
         self.hidden_size, self.eps, self.gain_name = hidden_size, float(eps), gain_name
         self.dtype, self.device = dtype, device
         self.branches = [(name, build_part("mixer", spec, dtype, device)) for name, spec in branches]
@@ -42,8 +51,11 @@ class ParallelMixer(Mixer):
             out += m.work_keys()
         return out
 
+    def paged_work(self, cache):
+        return [key for name, m in self.branches for key in m.paged_work(cache.sub[name])]
+
     def kernel_libraries(self, dtype):
-        out = [("streams", None)]
+        out = [("streams", None)] if self.combine == "rms_mean" else []
         for _, m in self.branches:
             out += m.kernel_libraries(dtype)
         return out
@@ -52,17 +64,21 @@ class ParallelMixer(Mixer):
         out = []
         for name, m in self.branches:
             out += m.param_specs(prefix + name + ".")
-            out.append(ParamSpec(prefix + name + "." + self.gain_name, (self.hidden_size,)))
+            if self.combine == "rms_mean":
+                out.append(ParamSpec(prefix + name + "." + self.gain_name, (self.hidden_size,)))
         return out
 
     def load(self, tensors, prefix):
         self.gains = []
         for name, m in self.branches:
             m.load(tensors, prefix + name + ".")
-            self.gains.append(tensors.pop(prefix + name + "." + self.gain_name).to(torch.float32).contiguous())
+            if self.combine == "rms_mean":
+                self.gains.append(tensors.pop(prefix + name + "." + self.gain_name).to(torch.float32).contiguous())
 
     def forward(self, x, ctx, cache):
         outs = [m.forward(x, ctx, cache.sub[name]) for name, m in self.branches]
+        if self.combine == "sum":
+            return DeltaSum(outs[0], outs[1] if len(outs) > 1 else None, self.scales[0], self.scales[-1])
         return ops.branch_rms_mean(outs, self.gains, self.eps)
 
 
