@@ -1,14 +1,16 @@
 #!/usr/bin/env python3
 """A design beside the engine's closest existing model at equal layer sizes (random weights).
 
-    python bench.py --design gebadra|bavetar|gusorax|mobunex|tuterax [--steps K] [--warmup W] [--sizes 2048,4096]
+    python bench.py --design gebadra|bavetar|gusorax|mobunex|tuterax|malilorn [--steps K] [--warmup W] [--sizes 2048,4096]
 
 For each size: prefill (one 2,048-token prompt in one step) and decode (batch 8 from 2,048-token
 contexts, the captured decode step) throughput of a few layers of the design and of a Qwen2 model
 with the same width, heads, key/value heads, feed-forward width, vocabulary and number of
 layers (Mobunex stands beside Bavetar, the engine's closest model: latent attention, a recurrent
 layer behind a short convolution, routed experts; Tuterax beside Mobunex - the same masked attention, a
-norm launch per sublayer - and Bavetar - a matrix state per head behind a short convolution); and the device time of the design's own kernels in one prompt step and one decode step,
+norm launch per sublayer - and Bavetar - a matrix state per head behind a short convolution; Malilorn
+beside Tuterax - the same attention, a matrix state per head with a decay per key channel - and Mobunex -
+routed and shared experts); and the device time of the design's own kernels in one prompt step and one decode step,
 each beside the like kernel of the Qwen2 model, with the fraction of its roofline (the slower of
 algorithmic bytes over the measured copy bandwidth and algorithmic FLOPs over the measured bf16
 GEMM rate).  Times are CUDA events on the launching stream after warm-up; the per-kernel times
@@ -108,6 +110,21 @@ def tuterax_config(width: int) -> dict:
               dict(type="attention", mixer=att, mlp=dense), dict(type="delta", mixer=delta, mlp=None)][:LAYERS]
     return dict(architecture="Tuterax", width=width, vocab=32000, norm=dict(eps=1e-6),
                 embedding=dict(scale=float(width) ** 0.5), layers=layers)
+
+
+def malilorn_config(width: int) -> dict:
+    """Four layers at the sizes of a real model of this kind: attention with heads of 128 (half of each turned,
+    slow pairs stretched), an eighth as many key/value heads and 4 taps; time mixing with as many heads of 128
+    as fill the width; a dense feed-forward twice and, twice, 32 experts of a quarter of its width, of which 4
+    are chosen, with a shared expert of the same width."""
+    heads, ff = width // 128, {2048: 5632, 4096: 11008}.get(width, width * 11 // 4)
+    left = dict(heads=heads, kv_heads=max(1, heads // 8), dim=128, vdim=128, conv=4, scale=128 ** -0.5,
+                rot=dict(base=1000000.0, dims=64, scaling=dict(factor=8.0, low=1.0, high=4.0, original=4096)))
+    mixer = dict(left=left, right=dict(heads=heads, dim=128), left_scale=1.0, right_scale=0.7)
+    dense = dict(kind="dense", ff=ff)
+    moe = dict(kind="moe", expert=dict(ff=ff // 4), router=dict(experts=32, top=4), shared=dict(ff=ff // 4))
+    layers = [dict(type="parallel", mixer=mixer, mlp=m) for m in (dense, moe, dense, moe)][:LAYERS]
+    return dict(architecture="Malilorn", width=width, vocab=32000, norm=dict(eps=1e-6), logit_softcap=30.0, layers=layers)
 
 
 def qwen_config(width: int, design: str = "gebadra") -> dict:
@@ -416,6 +433,64 @@ def rooflines_tuterax(width: int, pk: dict):
     return out
 
 
+def rooflines_malilorn(width: int, pk: dict):
+    """Algorithmic bytes and FLOPs of the compared kernels for the two workloads, per launch."""
+    c = malilorn_config(width)
+    a, t = c["layers"][0]["mixer"]["left"], c["layers"][0]["mixer"]["right"]
+    H, G, D, E, taps = a["heads"], a["kv_heads"], a["dim"], a["vdim"], a["conv"]
+    RH, RD = t["heads"], t["dim"]
+    rank = 32                                 # what random weights are made with
+    ff = c["layers"][0]["mlp"]["ff"]
+    r = c["layers"][1]["mlp"]
+    NE, top, eff = r["router"]["experts"], r["router"]["top"], r["expert"]["ff"]
+    T, R, Cx = PROMPT, BATCH, PROMPT
+
+    def t_us(by, fl):
+        return max(by / (pk["hbm_gbs"] * 1e9), fl / (pk["bf16_tflops"] * 1e12)) * 1e6
+
+    def both(rows, keys_total, keys_read, requests):
+        proj = (H * D + G * (D + E)) * 2
+        pairs = rows * top
+        # the last norm of a step reads the wanted rows only; a mixer's norm reads two branches, a feed-forward's one
+        norms = [rows * width * (2 * n + 4 + 4 + 2) for n in (2, 1) for _ in c["layers"]]
+        norms[-1] = requests * width * (2 + 4 + 2)
+        return {
+            "norm_add_norm": t_us(sum(norms) / len(norms), 0),
+            "head_conv_norm_write": t_us(rows * (proj + 4 * H * D + 2 * G * (D + E))
+                                         + 8 * requests * (taps - 1) * (H * D + G * (D + E)), 0),
+            "masked_attention": t_us(4 * rows * H * D + 2 * keys_read * G * (D + E) + 2 * rows * H * E,
+                                     2 * H * (D + E) * keys_total),
+            "token_shift": t_us(rows * width * 2 * 6, 0),
+            "linear_groups": t_us(4 * (2 * rows * width + 2 * width * RH * RD + 2 * rows * RH * RD),
+                                  8 * rows * width * RH * RD),
+            "low_rank_decay": t_us(rows * (4 * rank + 4 * RH * RD) + 2 * rank * RH * RD, 0),
+            "wkv": t_us(rows * RH * RD * (3 * 2 + 4 + 4) + 8 * requests * RH * RD * RD, 4 * rows * RH * RD * RD),
+            "gated_rms": t_us(rows * RH * RD * (4 + 2 + 2), 0),
+            "gated_activation": t_us(rows * ff * 6, 0),
+            "route": t_us(rows * (NE + 1) * 4, 0),
+            "expert_rows": t_us(2 * min(NE, pairs) * 2 * eff * width, 4 * pairs * eff * width),
+            "expert_gather": t_us(2 * rows * width + 2 * pairs * width, 0),
+            "expert_scatter": t_us(2 * pairs * width + 2 * rows * width * 2, 0),
+            # the mean over the up and down products
+            "grouped_runs": t_us(2 * pairs * (width + eff) + 2 * NE * eff * width, 2 * pairs * eff * width),
+        }
+    out = {"prefill": both(T, T * (T + 1) // 2, T, 1), "decode": both(R, R * (Cx + 1), R * (Cx + 1), R)}
+    m = mobunex_config(width)["layers"][1]["mlp"]
+    m_eff, m_pairs = m["expert"]["ff"], m["router"]["top"]
+    for beside, roofs in (("tuterax", rooflines_tuterax), ("mobunex", rooflines_mobunex)):
+        for phase in ("prefill", "decode"):
+            rows = T if phase == "prefill" else R
+            kernels = dict(roofs(width, pk)[phase])
+            if beside == "mobunex":           # its experts have gates: the mean over gate/up and down
+                pairs = rows * m_pairs
+                kernels["grouped_runs"] = t_us(2 * pairs * (width + 1.5 * m_eff) + 3 * m["router"]["experts"] * m_eff * width,
+                                               3 * pairs * m_eff * width)
+                kernels["expert_gather"] = t_us(2 * rows * width + 2 * pairs * width, 0)
+                kernels["expert_scatter"] = t_us(2 * pairs * width + 2 * rows * width * 2, 0)
+            out[f"{beside}.{phase}"] = kernels
+    return out
+
+
 def rooflines(width: int, pk: dict):
     """Algorithmic bytes and FLOPs of the compared kernels for the two workloads, per launch."""
     g = gebadra_config(width)
@@ -453,7 +528,7 @@ def run(design: str, steps: int, warmup: int, sizes=(2048, 4096)) -> dict:
     from bench import ClockSampler, peaks
     from paged_batch_engine_b200.config import load_config
     from paged_batch_engine_b200.engine.runner import ModelRunner
-    known = ("gebadra", "bavetar", "gusorax", "mobunex", "tuterax")
+    known = ("gebadra", "bavetar", "gusorax", "mobunex", "tuterax", "malilorn")
     if design not in known:
         raise SystemExit(f"unknown design {design!r}; known: {', '.join(known)}")
     os.environ["PBE_EXEC"] = "python"        # per-kernel times need every launch to come through ops
@@ -483,14 +558,20 @@ def run(design: str, steps: int, warmup: int, sizes=(2048, 4096)) -> dict:
     if design == "mobunex":
         own = mobunex_ops
         besides = [("bavetar", bavetar_config, bavetar_ops)]
+    tuterax_ops = ["norm_add", "embedding_positions", "head_norm_write", "masked_attention", "gated_activation",
+                   "delta_inputs", "delta_scan", "gated_rms"]
+    if design == "malilorn":
+        own = ["norm_add_norm", "head_conv_norm_write", "masked_attention", "token_shift", "linear_groups",
+               "low_rank_decay", "wkv", "gated_rms", "gated_activation", "route", "expert_rows", "expert_places",
+               "expert_gather", "expert_scatter", "grouped_runs", "run_tiles", "relu_squared"]
+        besides = [("tuterax", tuterax_config, tuterax_ops), ("mobunex", mobunex_config, mobunex_ops)]
     if design == "tuterax":
-        own = ["norm_add", "embedding_positions", "head_norm_write", "masked_attention", "gated_activation",
-               "delta_inputs", "delta_scan", "gated_rms"]
+        own = tuterax_ops
         besides = [("mobunex", mobunex_config, mobunex_ops), ("bavetar", bavetar_config, bavetar_ops)]
     design_config = {"bavetar": bavetar_config, "gusorax": gusorax_config, "mobunex": mobunex_config,
-                     "tuterax": tuterax_config}.get(design, gebadra_config)
+                     "tuterax": tuterax_config, "malilorn": malilorn_config}.get(design, gebadra_config)
     roofs = {"bavetar": rooflines_bavetar, "gusorax": rooflines_gusorax, "mobunex": rooflines_mobunex,
-             "tuterax": rooflines_tuterax}.get(design, rooflines)
+             "tuterax": rooflines_tuterax, "malilorn": rooflines_malilorn}.get(design, rooflines)
     sampler = ClockSampler(0)
     sampler.active = True
     out = {}

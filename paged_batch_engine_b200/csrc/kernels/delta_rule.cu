@@ -544,7 +544,7 @@ int launch_chunks(const ChunkParams& g, const ChunkScanParams<float>& p, int rec
   if (!opted) {
     cudaFuncSetAttribute(delta_chunks_kernel<DP, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_g);
     cudaFuncSetAttribute(delta_chunks_kernel<DP, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_g);
-    const cudaError_t e = cudaFuncSetAttribute(scan_chunks_kernel<RPT, CPT, WARPS, true, float>,
+    const cudaError_t e = cudaFuncSetAttribute(scan_chunks_kernel<RPT, CPT, WARPS, true, false, float>,
                                                cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_p);
     if (e != cudaSuccess) return (int)e;
     opted = true;
@@ -554,7 +554,7 @@ int launch_chunks(const ChunkParams& g, const ChunkScanParams<float>& p, int rec
   else launch_k(delta_chunks_kernel<DP, false>, grid, 128, smem_g, stream, g);
   const int err = launch_status();
   if (err != 0) return err;
-  launch_spread(scan_chunks_kernel<RPT, CPT, WARPS, true, float>, dim3(g.R, g.H, (g.E + COLS - 1) / COLS), 32 * WARPS, smem_p,
+  launch_spread(scan_chunks_kernel<RPT, CPT, WARPS, true, false, float>, dim3(g.R, g.H, (g.E + COLS - 1) / COLS), 32 * WARPS, smem_p,
                 stream, p);
   return launch_status();
 }

@@ -39,6 +39,8 @@ struct SkinnyParams {
   int n_out;          // row stride of Y: N (plain) or N / 2 (SwiGLU)
   int glu;            // the gated epilogue's activation: 0 silu, 1 gelu (tanh form), 2 relu; the plain one's: 3 relu squared
   int tiles;          // 16-row tiles (plain: ceil(N/16); SwiGLU: ceil((N/2)/8))
+  // products side by side (blockIdx.y): group g reads X + g M K and W + g N K and writes Y + g M n_out
+  int groups = 1;
 };
 
 __device__ __forceinline__ void mma_bf16(float (&c)[4], unsigned a0, unsigned a1, unsigned a2, unsigned a3,
@@ -102,6 +104,12 @@ template <int NT, int WARPS, bool SHORT = false> struct Stages {
 template <int NT, int WN, int WK, int CL, bool SWIGLU, typename TY, bool SHORT = false>
 __global__ void __launch_bounds__(WN * WK * 32)
 gemm_skinny_kernel(SkinnyParams p) {
+  if (p.groups > 1) {
+    const size_t grp = blockIdx.y;
+    p.X += grp * p.M * p.K;
+    p.W += grp * p.N * p.K;
+    p.Y = (TY*)p.Y + grp * p.M * p.n_out;
+  }
   constexpr int STAGES = Stages<NT, WN * WK, SHORT>::value;
   constexpr int SLOT = 2 + NT;                       // 16-byte chunks per thread and stage
   extern __shared__ __align__(16) uint4 ring[];      // [WN * WK][STAGES][SLOT][32]
@@ -277,8 +285,8 @@ int launch_cfg(const SkinnyParams& p, int row_blocks, cudaStream_t stream) {
                          cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     opted = true;
   }
-  launch_k_cluster(gemm_skinny_kernel<NT, WN, WK, CL, SWIGLU, TY, SHORT>, row_blocks * CL, WN * WK * 32, smem, stream,
-                   CL, p);
+  launch_k_cluster(gemm_skinny_kernel<NT, WN, WK, CL, SWIGLU, TY, SHORT>, dim3(row_blocks * CL, p.groups), WN * WK * 32,
+                   smem, stream, CL, p);
   return launch_status();
 }
 
@@ -299,8 +307,8 @@ PBE_EXPORT int pbe_gemm_skinny_max_rows() { return 16; }
 
 // mode 0: plain; 1: SwiGLU over a [gate; up] weight (N even, Y is [M, N/2]); 3: the same with gelu (tanh form);
 // 5: with relu; 4: plain, the result's relu squared.
-PBE_EXPORT int pbe_gemm_skinny(const void* X, const void* W, const float* bias, void* Y, int y_dtype,
-                               int M, int N, int K, int mode, cudaStream_t stream) {
+static int skinny(const void* X, const void* W, const float* bias, void* Y, int y_dtype, int M, int N, int K, int mode,
+                  int groups, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (M > 16 || K <= 0 || (K & 7) != 0) return (int)cudaErrorInvalidValue;
   const int glu = mode == 3 ? 1 : mode == 5 ? 2 : mode == 4 ? 3 : 0;
@@ -309,6 +317,7 @@ PBE_EXPORT int pbe_gemm_skinny(const void* X, const void* W, const float* bias, 
   if (mode == 1 && (N & 1)) return (int)cudaErrorInvalidValue;
   SkinnyParams p;
   p.glu = glu;
+  p.groups = groups;
   p.X = (const bf16*)X;
   p.W = (const bf16*)W;
   p.bias = bias;
@@ -328,4 +337,16 @@ PBE_EXPORT int pbe_gemm_skinny(const void* X, const void* W, const float* bias, 
   if (M <= 8) GO(1);
   GO(2);
 #undef GO
+}
+
+PBE_EXPORT int pbe_gemm_skinny(const void* X, const void* W, const float* bias, void* Y, int y_dtype,
+                               int M, int N, int K, int mode, cudaStream_t stream) {
+  return skinny(X, W, bias, Y, y_dtype, M, N, K, mode, 1, stream);
+}
+
+// `groups` plain products of equal sizes side by side: X [groups, M, K], W [groups, N, K], Y [groups, M, N].
+PBE_EXPORT int pbe_gemm_skinny_groups(const void* X, const void* W, void* Y, int y_dtype, int M, int N, int K,
+                                      int groups, cudaStream_t stream) {
+  if (groups < 1 || groups > 65535) return (int)cudaErrorInvalidValue;
+  return skinny(X, W, nullptr, Y, y_dtype, M, N, K, 0, groups, stream);
 }

@@ -332,25 +332,59 @@ __global__ void __launch_bounds__(128) wkv_chunks_kernel(WkvParams p, float* rec
   }
 }
 
+// How long portions are cut into segments (all null: they are not)
+struct Segments {
+  const int32_t* first;      // [n_first, 4] the segments whose own contributions are needed
+  int n_first;
+  const int32_t* starts;     // [n_starts, 4]
+  int n_starts;
+  const int32_t* second;     // [n_second, 4] every segment, and the requests that are not cut
+  int n_second;
+  float* scratch;            // [entries, H, E, D]
+  float* own_decay;          // [entries, H, D]
+  const int32_t* request_of_row;
+};
+
 template <typename T, int RPT, int CPT, int WARPS>
-int launch_chunks(const WkvParams& g, float* records, int count, cudaStream_t stream) {
+int launch_chunks(const WkvParams& g, float* records, int count, const Segments& s, cudaStream_t stream) {
   constexpr int DP = 16 * RPT, COLS = 2 * WARPS * CPT;
   constexpr size_t smem_g = sizeof(float) * 3 * CH * DP, smem_p = sizeof(float) * 2 * record_floats(DP, false);
   static bool opted = false;
   if (!opted) {
     cudaFuncSetAttribute(wkv_chunks_kernel<T, DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_g);
-    const cudaError_t e = cudaFuncSetAttribute(scan_chunks_kernel<RPT, CPT, WARPS, false, T>,
+    cudaFuncSetAttribute(scan_chunks_kernel<RPT, CPT, WARPS, false, true, T>,
+                         cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_p);
+    const cudaError_t e = cudaFuncSetAttribute(scan_chunks_kernel<RPT, CPT, WARPS, false, false, T>,
                                                cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_p);
     if (e != cudaSuccess) return (int)e;
     opted = true;
   }
   launch_k(wkv_chunks_kernel<T, DP>, dim3(count, g.H), 128, smem_g, stream, g, records);
-  const int err = launch_status();
+  int err = launch_status();
   if (err != 0) return err;
-  const ChunkScanParams<T> p{records, (const T*)g.v, g.ld_v, g.out, g.state, g.q_start, g.q_len, g.slots,
-                             g.H, g.D, g.E, g.write_state};
-  launch_spread(scan_chunks_kernel<RPT, CPT, WARPS, false, T>, dim3(g.R, g.H, (g.E + COLS - 1) / COLS), 32 * WARPS,
-                smem_p, stream, p);
+  ChunkScanParams<T> p{records, (const T*)g.v, g.ld_v, g.out, g.state, g.q_start, g.q_len, g.slots,
+                       g.H, g.D, g.E, g.write_state};
+  const int slices = (g.E + COLS - 1) / COLS;
+  if (s.second == nullptr) {
+    launch_spread(scan_chunks_kernel<RPT, CPT, WARPS, false, false, T>, dim3(g.R, g.H, slices), 32 * WARPS, smem_p,
+                  stream, p);
+    return launch_status();
+  }
+  p.scratch = s.scratch;
+  p.own_decay = s.own_decay;
+  p.request_of_row = s.request_of_row;
+  p.items = s.first;
+  launch_spread(scan_chunks_kernel<RPT, CPT, WARPS, false, true, T>, dim3(s.n_first, g.H, slices), 32 * WARPS, smem_p,
+                stream, p);
+  err = launch_status();
+  if (err != 0) return err;
+  launch_k(segment_starts_kernel, dim3(s.n_starts, g.H, (unsigned)(((size_t)g.D * g.E + 255) / 256)), 256, 0, stream,
+           (const float*)g.state, s.scratch, (const float*)s.own_decay, s.starts, g.H, g.D, g.E);
+  err = launch_status();
+  if (err != 0) return err;
+  p.items = s.second;
+  launch_spread(scan_chunks_kernel<RPT, CPT, WARPS, false, false, T>, dim3(s.n_second, g.H, slices), 32 * WARPS, smem_p,
+                stream, p);
   return launch_status();
 }
 
@@ -429,22 +463,29 @@ PBE_EXPORT int pbe_wkv_record_floats(int D) {
 PBE_EXPORT int pbe_wkv_chunk_tokens() { return CH; }
 
 // The same for steps with prompt portions, sixteen tokens of a request at a time: two launches.
-// records: [T / 16 + R][H][pbe_wkv_record_floats(D)] floats of scratch memory.
+// records: [T / 16 + R][H][pbe_wkv_record_floats(D)] floats of scratch memory.  With `second` (segments of whole
+// chunks, see chunk_scan.cuh) long portions run as segments side by side: two launches more.
 PBE_EXPORT int pbe_wkv_chunks(const void* r, const void* k, const void* v, int ld_r, int ld_k, int ld_v, int dtype,
                               const float* decay, const float* bonus, float* out, float* state, float* records,
                               const int32_t* q_start, const int32_t* q_len, const int32_t* slots, int T, int R, int H,
-                              int D, int E, int write_state, cudaStream_t stream) {
+                              int D, int E, int write_state, const int32_t* first, int n_first, const int32_t* starts,
+                              int n_starts, const int32_t* second, int n_second, float* scratch, float* own_decay,
+                              const int32_t* request_of_row, cudaStream_t stream) {
   if (R <= 0 || T <= 0) return 0;
+  if (second != nullptr && (!first || !starts || !scratch || !own_decay || !request_of_row || n_first < 1 || n_starts < 1))
+    return (int)cudaErrorInvalidValue;
+  if (((uintptr_t)scratch & 15) != 0) return (int)cudaErrorMisalignedAddress;
+  const Segments s{first, n_first, starts, n_starts, second, n_second, scratch, own_decay, request_of_row};
   if (D < 1 || D > 256 || E < 1 || H < 1 || records == nullptr) return (int)cudaErrorInvalidValue;
   if ((((uintptr_t)state | (uintptr_t)records | (uintptr_t)decay) & 15) != 0) return (int)cudaErrorMisalignedAddress;
   WkvParams p{r, k, v, ld_r, ld_k, ld_v, decay, bonus, out, state, q_start, q_len, slots, R, H, D, E, write_state};
   const int n = T / CH + R;
   if (dtype == PBE_F32) {
-    if (D <= 64) return launch_chunks<float, 4, 2, 4>(p, records, n, stream);
-    if (D <= 128) return launch_chunks<float, 8, 2, 4>(p, records, n, stream);
-    return launch_chunks<float, 16, 2, 4>(p, records, n, stream);
+    if (D <= 64) return launch_chunks<float, 4, 4, 4>(p, records, n, s, stream);
+    if (D <= 128) return launch_chunks<float, 8, 4, 4>(p, records, n, s, stream);
+    return launch_chunks<float, 16, 2, 4>(p, records, n, s, stream);
   }
-  if (D <= 64) return launch_chunks<__nv_bfloat16, 4, 2, 4>(p, records, n, stream);
-  if (D <= 128) return launch_chunks<__nv_bfloat16, 8, 2, 4>(p, records, n, stream);
-  return launch_chunks<__nv_bfloat16, 16, 2, 4>(p, records, n, stream);
+  if (D <= 64) return launch_chunks<__nv_bfloat16, 4, 4, 4>(p, records, n, s, stream);
+  if (D <= 128) return launch_chunks<__nv_bfloat16, 8, 4, 4>(p, records, n, s, stream);
+  return launch_chunks<__nv_bfloat16, 16, 2, 4>(p, records, n, s, stream);
 }

@@ -861,6 +861,31 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
     return torch.mm(x, w.t())
 
 
+def linear_groups(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """y[s] = x[s] w[s]^T for products of equal sizes with operands of their own: x [S, T, K], w [S, N, K]; returns
+    [S, T, N] in x's dtype.  Few rows take the package's weight-streaming kernel, all products in one launch;
+    many the library's batched product; a float32 weight the package's true-float32 kernel."""
+    _need_cuda(x, w)
+    _need_contiguous(x, w)
+    S, T, K = x.shape
+    N = w.shape[1]
+    if tuple(w.shape) != (S, N, K):
+        raise KernelError("linear_groups: x is [S, T, K], w [S, N, K]")
+    if w.dtype == torch.float32:
+        out = torch.empty((S, T, N), dtype=x.dtype, device=x.device)
+        for s in range(S):
+            sgemm_nt(x[s], w[s], None, out[s])
+        return out
+    if x.dtype != torch.bfloat16:
+        raise KernelError("a bfloat16 weight takes bfloat16 activations")
+    if 0 < T <= SKINNY_MAX_ROWS and K % 8 == 0:
+        out = torch.empty((S, T, N), dtype=torch.bfloat16, device=x.device)
+        fn = _fn("gemm_skinny", "pbe_gemm_skinny_groups", [c_void_p] * 3 + [c_int] * 5 + [c_void_p])
+        _check(fn(_ptr(x), _ptr(w), _ptr(out), BF16, T, N, K, S, _stream()), "gemm_skinny_groups")
+        return out
+    return torch.bmm(x, w.transpose(1, 2))
+
+
 # ------------------------------------------------------------------ attention
 class AttnParams(ctypes.Structure):
     _fields_ = [("q", c_void_p), ("k_cache", c_void_p), ("v_cache", c_void_p), ("out", c_void_p),
@@ -2291,12 +2316,15 @@ WKV_CHUNK_MAX_DIM = 256       # wider key heads always run token by token
 
 def wkv(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, bonus: torch.Tensor,
         state: torch.Tensor, q_start: torch.Tensor, q_len: torch.Tensor, slots: torch.Tensor, num_requests: int,
-        heads: int, update_state: bool = True, zero_out: bool = False, chunked: bool = False) -> torch.Tensor:
+        heads: int, update_state: bool = True, zero_out: bool = False, chunked: bool = False, plan=None,
+        request_of_row: Optional[torch.Tensor] = None) -> torch.Tensor:
     """o_t = (S + diag(bonus) k_t v_t^T)^T r_t, S <- diag(decay_t) S + k_t v_t^T per head, request by request over
     the rows each brings: ``r``, ``k`` [T, H * D] and ``v`` [T, H * E] column slices in one dtype, ``decay`` float32
     [T, H * D] (numbers in [0, 1]), ``bonus`` float32 [H * D], ``state`` float32 [slots, H, E, D] (S transposed: a
     value column's key channels side by side), read at ``slots[r]`` and left updated.  ``chunked``: sixteen
-    tokens at a time (prompt portions: two launches), else one by one.  Returns o, float32 [T, H * E]."""
+    tokens at a time (prompt portions: two launches), else one by one.  ``plan`` (a ``RecurrencePlan`` of the step
+    whose chunks are multiples of sixteen rows; with ``request_of_row`` int32 [T]): chunked portions of several
+    such lengths run as segments side by side (two launches more).  Returns o, float32 [T, H * E]."""
     _need_cuda(r, k, v, decay, bonus, state, q_start, q_len, slots)
     _need_contiguous(decay, bonus, state)
     for x in (r, k, v):
@@ -2326,11 +2354,21 @@ def wkv(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, 
         size = _fn("time_mixing", "pbe_wkv_record_floats", [c_int])(D)
         ct = _fn("time_mixing", "pbe_wkv_chunk_tokens", [])()
         records = torch.empty((T // ct + int(num_requests), H, size), dtype=torch.float32, device=v.device)
-        fn = _fn("time_mixing", "pbe_wkv_chunks", types + [c_void_p] * 4 + [c_int] * 6 + [c_void_p])
+        segments = [None, 0, None, 0, None, 0, None, None, None]
+        if plan is not None and plan.num_chunks > 0:
+            if request_of_row is None or plan.rows_per_chunk % ct:
+                raise KernelError("wkv: segments are whole chunks, and their rows' requests are needed")
+            scratch = torch.empty((plan.num_chunks, H, E, D), dtype=torch.float32, device=v.device)
+            own_decay = torch.empty((plan.num_chunks, H, D), dtype=torch.float32, device=v.device)
+            segments = [_ptr(plan.first_pass), plan.num_first_pass, _ptr(plan.scan), plan.num_scan,
+                        _ptr(plan.second_pass), plan.num_second_pass, _ptr(scratch), _ptr(own_decay),
+                        _ptr(request_of_row)]
+        fn = _fn("time_mixing", "pbe_wkv_chunks", types + [c_void_p] * 4 + [c_int] * 6 + [c_void_p, c_int] * 3
+                 + [c_void_p] * 4)
         global _launches
         _check(fn(*heads_of, _ptr(records), _ptr(q_start), _ptr(q_len), _ptr(slots), T, int(num_requests), H, D, E,
-                  1 if update_state else 0, _stream()), "wkv_chunks")
-        _launches += 1
+                  1 if update_state else 0, *segments, _stream()), "wkv_chunks")
+        _launches += 1 if segments[4] is None else 3
         return out
     fn = _fn("time_mixing", "pbe_wkv_steps", types + [c_void_p] * 3 + [c_int] * 5 + [c_void_p])
     _check(fn(*heads_of, _ptr(q_start), _ptr(q_len), _ptr(slots), int(num_requests), H, D, E, 1 if update_state else 0,

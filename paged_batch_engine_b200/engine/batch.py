@@ -229,6 +229,7 @@ class RecurrencePlan:
     num_scan: int = 0
     second_pass: Optional[torch.Tensor] = None
     num_second_pass: int = 0
+    rows_per_chunk: int = 0
 
 
 def recurrence_plan_arrays(q_start, q_len, slots, chunk: int):
@@ -383,7 +384,8 @@ class StepContext:
                     host = host.pin_memory()
                 dev = host.to(self.device, non_blocking=True)
                 a, b = len(first), len(first) + len(scan)
-                plan = RecurrencePlan(entries, dev[:a], a, dev[a:b], len(scan), dev[b:], len(second))
+                plan = RecurrencePlan(entries, dev[:a], a, dev[a:b], len(scan), dev[b:], len(second),
+                                      rows_per_chunk=chunk)
                 self.__dict__.setdefault("_plan_hosts", []).append(host)     # pinned until the step is done
             plans[chunk] = plan
         return plan

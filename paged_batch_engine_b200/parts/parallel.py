@@ -1,6 +1,7 @@
 """Several mixers side by side on the same input."""
 from __future__ import annotations
 
+import os
 from typing import Optional, Sequence, Tuple
 
 import torch
@@ -10,6 +11,9 @@ from ..csrc import ops
 from ..weights.loader import ParamSpec
 from .base import CompositeNeed, Mixer, build_part, register_part
 from .norm import DeltaSum
+
+# PBE_BRANCHES=serial keeps a captured step's branches one after the other
+SIDE_BY_SIDE = os.environ.get("PBE_BRANCHES", "").strip().lower() != "serial"
 
 
 class ParallelMixer(Mixer):
@@ -75,8 +79,35 @@ class ParallelMixer(Mixer):
             if self.combine == "rms_mean":
                 self.gains.append(tensors.pop(prefix + name + "." + self.gain_name).to(torch.float32).contiguous())
 
+    _side_streams = {}        # (device, branch) -> the stream a branch is recorded on
+
+    def _side_by_side(self, x, ctx, cache):
+        main = torch.cuda.current_stream()
+        fork = torch.cuda.Event()
+        fork.record(main)
+        outs = [None] * len(self.branches)
+        for i, (name, m) in enumerate(self.branches[1:], start=1):
+            side = self._side_streams.get((x.device, i))
+            if side is None:
+                side = self._side_streams[(x.device, i)] = torch.cuda.Stream(device=x.device)
+            side.wait_event(fork)
+            with torch.cuda.stream(side):
+                outs[i] = m.forward(x, ctx, cache.sub[name])
+                join = torch.cuda.Event()
+                join.record(side)
+            outs[i] = (outs[i], join)
+        name, m = self.branches[0]
+        outs[0] = m.forward(x, ctx, cache.sub[name])
+        for i in range(1, len(outs)):
+            outs[i], join = outs[i]
+            main.wait_event(join)
+        return outs
+
     def forward(self, x, ctx, cache):
-        outs = [m.forward(x, ctx, cache.sub[name]) for name, m in self.branches]
+        if SIDE_BY_SIDE and len(self.branches) > 1 and getattr(ctx, "captured", False):
+            outs = self._side_by_side(x, ctx, cache)
+        else:
+            outs = [m.forward(x, ctx, cache.sub[name]) for name, m in self.branches]
         if self.combine == "sum":
             return DeltaSum(outs[0], outs[1] if len(outs) > 1 else None, self.scales[0], self.scales[-1])
         return ops.branch_rms_mean(outs, self.gains, self.eps)

@@ -68,7 +68,12 @@ class TimeMixing(Mixer):
         n = self.names
         f32 = lambda name: tensors.pop(prefix + name).to(torch.float32).contiguous()
         self.mu = torch.stack([f32(n["mu"] + n[s]) for s in self.BLENDS]).contiguous()      # [5, hidden]
-        self.w_in = [tensors.pop(prefix + n[s]).contiguous() for s in "rkvg"]
+        ws = [tensors.pop(prefix + n[s]) for s in "rkvg"]
+        if len({w.dtype for w in ws}) != 1:
+            ws = [w.to(torch.float32) for w in ws]
+        # products of equal sizes are one launch: r, k, v and the gate together, or the pairs
+        self.w_in = [torch.stack(ws)] if self.key_dim == self.value_dim else [torch.stack(ws[:2]), torch.stack(ws[2:])]
+        del ws
         self.w_low = tensors.pop(prefix + n["w1"]).contiguous()
         w2 = tensors.pop(prefix + n["w2"])
         if w2.shape[1] != self.w_low.shape[0]:
@@ -79,17 +84,32 @@ class TimeMixing(Mixer):
         self.w_o = tensors.pop(prefix + n["o"]).contiguous()
 
     # ---- compute
+    def segment_rows(self, rows: int) -> int:
+        """Rows of a segment when a long portion's recurrence is cut to run side by side: so long that the
+        segments of all heads and column slices fill the GPU a few times over, a power of two, 64 to 1,024."""
+        want = rows * self.num_heads * ((self.value_dim + 31) // 32) // 1024
+        segment = 64
+        while segment < want and segment < 1024:
+            segment *= 2
+        return segment
+
     def forward(self, x, ctx, cache):
         H = self.num_heads
         captured = getattr(ctx, "captured", False)
         single = captured or ctx.num_tokens == ctx.num_requests        # every request brings one token
         blends = ops.token_shift(x, self.mu, cache.sub["shift"].state, ctx.request_of_row, ctx.q_start, ctx.q_len,
                                  ctx.state_slots, ctx.num_requests, update_state=cache.writes)
-        r, k, v, g = (ops.linear(blends[i], w, None, out_dtype=self.dtype, kind=1) for i, w in enumerate(self.w_in))
+        made, first = [], 0
+        for w in self.w_in:
+            made += list(ops.linear_groups(blends[first:first + w.shape[0]], w).unbind(0))
+            first += w.shape[0]
+        r, k, v, g = made
         low = ops.linear(blends[4], self.w_low, None, out_dtype=torch.float32)
         decay = ops.low_rank_decay(low, self.w2_t, self.w0)
+        plan = None if single else ctx.recurrence_plan(self.segment_rows(ctx.num_tokens))
         o = ops.wkv(r, k, v, decay, self.bonus, cache.sub["wkv"].state, ctx.q_start, ctx.q_len, ctx.state_slots,
-                    ctx.num_requests, H, update_state=cache.writes, zero_out=captured, chunked=not single)
+                    ctx.num_requests, H, update_state=cache.writes, zero_out=captured, chunked=not single,
+                    plan=plan, request_of_row=ctx.request_of_row)
         y = ops.gated_rms(o, g, self.gain, H, self.eps, True, "silu", self.dtype)
         return ops.linear(y, self.w_o, None, out_dtype=self.dtype, kind=2)
 
