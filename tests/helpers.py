@@ -547,3 +547,100 @@ def make_tuterax_folder(path, cfg: dict, seed: int, dtype=torch.bfloat16, gain: 
         w[k] = t.to(w[k].dtype).contiguous()
     save_file(w, f)
     return str(path)
+
+
+# ---------------------------------------------------------------- Malilorn
+def _mleft(heads, kv, dim, vdim, conv, rot_dims, base, scale, scaling=None):
+    rot = dict(dims=rot_dims, base=base)
+    if scaling:
+        rot["scaling"] = dict(zip(("factor", "low", "high", "original"), scaling))
+    return dict(heads=heads, kv_heads=kv, dim=dim, vdim=vdim, conv=conv, scale=scale, rot=rot)
+
+
+def _mlayer(left, heads, dim, left_scale, right_scale, mlp):
+    return dict(type="parallel", mlp=mlp, mixer=dict(left=left, right=dict(heads=heads, dim=dim), left_scale=left_scale,
+                                                     right_scale=right_scale))
+
+
+def _mroute(ff, experts, top, shared=None):
+    d = dict(kind="moe", expert=dict(ff=ff), router=dict(experts=experts, top=top))
+    if shared:
+        d["shared"] = dict(ff=shared)
+    return d
+
+
+# three query heads a key head, the whole head turns, pairs kept, blended and stretched; two experts of five and
+# a shared one; values narrower than keys with a rotation of one pair; a layer without feed-forward
+MAL_A = dict(
+    architecture="Malilorn", width=72, vocab=300, norm=dict(eps=1e-5), logit_softcap=25.0,
+    layers=[
+        _mlayer(_mleft(6, 2, 24, 40, 3, 24, 1000.0, 0.2, (8.0, 1.0, 4.0, 64)), 3, 16, 1.3, 0.6, dict(kind="dense", ff=88)),
+        _mlayer(_mleft(2, 2, 12, 6, 4, 2, 50.0, 0.4, (2.0, 2.0, 3.0, 900)), 2, 24, 0.5, 1.7, _mroute(20, 5, 2, 36)),
+        _mlayer(_mleft(3, 1, 16, 24, 2, 6, 30.0, 0.3), 1, 20, 1.0, 1.0, None),
+    ])
+# heads the tensor cores take in bfloat16; one tap (no convolution state); as many key heads as heads; every
+# expert chosen, no shared one; one expert of seven; one head that is wider than a chunk is long
+MAL_B = dict(
+    architecture="Malilorn", width=96, vocab=211, norm=dict(eps=1e-6), logit_softcap=12.0,
+    layers=[
+        _mlayer(_mleft(4, 1, 32, 16, 1, 16, 300.0, 0.25, (4.0, 1.0, 4.0, 128)), 1, 40, 0.8, 1.1, _mroute(24, 3, 3)),
+        _mlayer(_mleft(5, 5, 16, 32, 3, 8, 5000.0, 0.3, (3.0, 0.5, 8.0, 256)), 4, 8, 1.2, 0.7, _mroute(40, 7, 1, 16)),
+        _mlayer(_mleft(2, 1, 48, 80, 6, 48, 100000.0, 0.15, (16.0, 1.0, 2.0, 512)), 2, 64, 1.0, 0.9,
+                dict(kind="dense", ff=72)),
+    ])
+# wide values; more than 64 key channels a state; widths no vector access divides; four experts of thirty-three;
+# no cap on the logits
+MAL_C = dict(
+    architecture="Malilorn", width=128, vocab=257, norm=dict(eps=1e-6), logit_softcap=None,
+    layers=[
+        _mlayer(_mleft(4, 1, 64, 128, 5, 32, 100000.0, 0.12, (4.0, 1.0, 4.0, 300)), 2, 72, 1.1, 0.9, _mroute(32, 33, 4, 48)),
+        _mlayer(_mleft(3, 3, 17, 9, 3, 10, 20.0, 0.3), 3, 33, 0.7, 1.4, dict(kind="dense", ff=50)),
+        _mlayer(_mleft(2, 1, 112, 16, 2, 64, 1000.0, 0.1, (2.0, 1.0, 1.0, 100)), 5, 7, 0.9, 0.9, _mroute(17, 6, 2, 9)),
+    ])
+MALILORN = {"A": (MAL_A, 91, 8), "B": (MAL_B, 92, 16), "C": (MAL_C, 93, 4)}     # config, seed, page tokens
+
+
+def make_malilorn_folder(path, cfg: dict, seed: int, dtype=torch.bfloat16, gain: float = 1.0, rank: int = 13) -> str:
+    """A model folder with seeded random weights through the engine's random-weights mode, then
+    reshaped so that no mechanism is a near-identity: norm gains far from one, sharp softmaxes,
+    convolutions with weight on every tap, blends from all of the row to all of the one before, decays
+    from almost nothing to almost one, biases and router scores spread over their range, a low rank
+    that is no multiple of eight.  ``gain`` scales the matrices' factors (wide models need less)."""
+    from paged_batch_engine_b200.config import load_config
+    from paged_batch_engine_b200.engine.runner import build_model
+    from paged_batch_engine_b200.weights import write_random_model
+    from safetensors.torch import load_file, save_file
+    _, typed = load_config(cfg)
+    model = build_model(typed, torch.float32, "cpu")
+    write_random_model(str(path), typed, model.param_specs(), seed, dtype)
+    f = os.path.join(str(path), "model.safetensors")
+    w = load_file(f)
+    g = torch.Generator().manual_seed(seed)
+    for k in list(w):
+        t = w[k].float()
+        leaf = k.split(".mix.")[-1] if ".mix." in k else k.split(".")[-1]
+        if k == "embed":
+            t = t * 25.0
+        elif leaf.startswith("norm") or k == "final.norm" or leaf.endswith(".norm"):
+            t = 0.4 + 1.4 * torch.rand(t.shape, generator=g)
+        elif leaf.endswith(".conv"):
+            t = torch.randn(t.shape, generator=g) * 0.6
+        elif ".mu." in leaf:
+            t = torch.rand(t.shape, generator=g)
+        elif leaf == "right.w0":
+            t = torch.randn(t.shape, generator=g) * 1.5 - 1.5
+        elif leaf == "right.u":
+            t = torch.randn(t.shape, generator=g)
+        elif leaf == "right.w1":
+            t = t[:rank] * 6.0 * gain
+        elif leaf == "right.w2":
+            t = t[:, :rank] * 25.0
+        elif k.endswith(".b"):
+            t = torch.randn(t.shape, generator=g) * 0.5
+        elif leaf in ("router", "sg"):
+            t = t * 8.0 * gain
+        elif t.dim() == 2:
+            t = t * 6.0 * gain
+        w[k] = t.to(w[k].dtype).contiguous()
+    save_file(w, f)
+    return str(path)
