@@ -116,7 +116,7 @@ def test_blocks_refuse_norms_and_residuals_they_cannot_use():
     with pytest.raises(TypeError, match="DepthStack"):
         good.forward(torch.zeros(2, 72), None, None, None)
     with pytest.raises(ValueError, match="activation"):
-        SwiGLU(8, 8, torch.float32, "cpu", activation="relu")
+        SwiGLU(8, 8, torch.float32, "cpu", activation="elu")
     common = dict(hidden_size=8, num_heads=2, num_kv_heads=1, key_dim=8, value_dim=8, scale=1.0, eps=1e-5,
                   dtype=torch.float32, device="cpu")
     with pytest.raises(ValueError, match="one sink"):
