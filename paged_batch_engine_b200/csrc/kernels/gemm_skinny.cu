@@ -101,10 +101,10 @@ template <int NT, int WARPS, bool SHORT = false> struct Stages {
 // STAGES-1 blocks ahead; a thread only ever reads the slots it filled itself, so the main
 // loop needs no barrier.  The first STAGES-1 weight blocks are requested before the
 // programmatic dependency on the previous kernel is awaited: weights do not depend on it.
-template <int NT, int WN, int WK, int CL, bool SWIGLU, typename TY, bool SHORT = false>
+template <int NT, int WN, int WK, int CL, bool SWIGLU, typename TY, bool SHORT = false, bool GROUPS = false>
 __global__ void __launch_bounds__(WN * WK * 32)
 gemm_skinny_kernel(SkinnyParams p) {
-  if (p.groups > 1) {
+  if constexpr (GROUPS) {
     const size_t grp = blockIdx.y;
     p.X += grp * p.M * p.K;
     p.W += grp * p.N * p.K;
@@ -276,16 +276,16 @@ gemm_skinny_kernel(SkinnyParams p) {
   }
 }
 
-template <int NT, int WN, int WK, int CL, bool SWIGLU, typename TY, bool SHORT = false>
+template <int NT, int WN, int WK, int CL, bool SWIGLU, typename TY, bool SHORT = false, bool GROUPS = false>
 int launch_cfg(const SkinnyParams& p, int row_blocks, cudaStream_t stream) {
   constexpr size_t smem = sizeof(uint4) * WN * WK * Stages<NT, WN * WK, SHORT>::value * (2 + NT) * 32;
   static bool opted = false;
   if (!opted) {
-    cudaFuncSetAttribute(gemm_skinny_kernel<NT, WN, WK, CL, SWIGLU, TY, SHORT>,
+    cudaFuncSetAttribute(gemm_skinny_kernel<NT, WN, WK, CL, SWIGLU, TY, SHORT, GROUPS>,
                          cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     opted = true;
   }
-  launch_k_cluster(gemm_skinny_kernel<NT, WN, WK, CL, SWIGLU, TY, SHORT>, dim3(row_blocks * CL, p.groups), WN * WK * 32,
+  launch_k_cluster(gemm_skinny_kernel<NT, WN, WK, CL, SWIGLU, TY, SHORT, GROUPS>, dim3(row_blocks * CL, p.groups), WN * WK * 32,
                    smem, stream, CL, p);
   return launch_status();
 }
@@ -297,6 +297,9 @@ int launch(const SkinnyParams& p, cudaStream_t stream) {
   // O, down): one row tile by four K slices, four warps a block, no cluster (a cluster of two
   // that splits K eight ways was slower by 10 % alone and equal in the step).
   const int tiles = p.tiles;
+  if constexpr (!SWIGLU) {
+    if (p.groups > 1) return launch_cfg<NT, 1, 4, 1, false, TY, false, true>(p, tiles, stream);
+  }
   if (tiles >= 148 * 8) return launch_cfg<NT, 2, 4, 1, SWIGLU, TY>(p, (tiles + 1) / 2, stream);
   if (NT == 1 && p.K <= 4096 && p.M == 1) return launch_cfg<NT, 1, 4, 1, SWIGLU, TY, true>(p, tiles, stream);
   return launch_cfg<NT, 1, 4, 1, SWIGLU, TY>(p, tiles, stream);
