@@ -101,6 +101,8 @@ __global__ void route_kernel(RouteParams p) {
   for (int i = 0; i < MAX_PER_LANE; ++i) {
     const int e = lane + 32 * i;
     c[i] = s[i] + ((p.correction && e < E) ? p.correction[e] : 0.f);
+    // plain sigmoid scores rank like their logits, which stay apart where the scores round to one or zero
+    if (p.score_kind == 1 && !p.correction && p.groups == 1 && e < E) c[i] = z[e] == z[e] ? z[e] : -INFINITY;
   }
   // allowed[i]: may expert lane + 32 i still be chosen
   bool allowed[MAX_PER_LANE];
